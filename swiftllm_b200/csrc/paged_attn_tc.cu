@@ -199,8 +199,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) paged_attn_tc_kernel(const __gr
         producer_loop<false>(p, &vmap, &qmap, v_sm, bars->v_full, bars->v_empty, TC_VSTAGES, bars, q_sm, g, lane);
     } else if (warp == 1) {
         // =========================================================== MMA issuer: two in-order queues, polled.  The whole warp
-        // runs the loop converged (votes keep the control flow provably uniform) and one elected lane issues, so ptxas keeps
-        // the UMMA descriptors in uniform registers instead of wrapping every UTCHMMA in a uniformisation loop.
+        // runs the loop converged (votes keep the control flow warp-uniform) and one elected lane issues (see elect_one).
         {
             constexpr uint32_t IDESC_S = make_instr_desc(128, TC_NPAD, UmmaFmt<T>::value, 0, 0);   // A K-major, B K-major
             constexpr uint32_t IDESC_O = make_instr_desc(128, TC_NPAD, UmmaFmt<T>::value, 1, 0);   // A MN-major (V^T)
