@@ -264,14 +264,15 @@ int sllm_latent_kv_store(const void* dkv, int64_t row_stride, const void* norm_w
 /* 16-bit dtypes with r % 16 == 0 and dr % 16 == 0 run on tensor cores (mma.sync over the heads of a token); other shapes and
  * SLLM_F32 run the fp32 CUDA-core kernel.  sllm_latent_attention_set_simt(1) forces the latter (returns the old setting). */
 int sllm_latent_attention_set_simt(int on);
-/* num_splits > 1 with split_workspace (fp32 [T, num_heads, num_splits, r + 2], device) lets the tensor-core kernel share a
+/* sink (fp32 [num_heads], or NULL): the softmax's denominator also contains exp(sink[h]) (no key, no value, not scaled).
+ * num_splits > 1 with split_workspace (fp32 [T, num_heads, num_splits, r + 2], device) lets the tensor-core kernel share a
  * query's visible keys between num_splits CTAs (steps with few tokens), merged by a second kernel; ignored by the other path. */
 int sllm_latent_attention(const void* q_lat, int64_t q_lat_stride_t, int64_t q_lat_stride_h, const void* q_rot,
                           int64_t q_rot_stride_t, int64_t q_rot_stride_h, const void* cosb, const void* sinb,
                           const void* gate, int64_t gate_stride_t, const void* cache, int n_slots, int slot, int block_size,
                           const void* block_table, int max_blocks_per_seq, const void* tok_seq, const void* tok_pos,
                           void* out, int64_t out_stride_t, int64_t out_stride_h, int64_t num_tokens, int num_heads, int r,
-                          int dr, int rot_dims, int window, float scale, int num_splits, void* split_workspace,
+                          int dr, int rot_dims, int window, float scale, const void* sink, int num_splits, void* split_workspace,
                           sllm_dtype_t dtype, sllm_stream_t stream);
 
 /* ---- Gated sliding-window attention with grouped key/value heads over a paged cache of per-token rows
@@ -302,7 +303,14 @@ int sllm_window_kv_store(const void* k, int64_t k_row_stride, const void* v, int
  * other shapes and SLLM_F32 run the fp32 CUDA-core kernel.  sllm_window_attention_set_simt(1) forces the latter (returns the
  * old setting).  softcap > 0: s_j <- softcap * tanh(s_j / softcap); out_scale multiplies the output.
  * chunk > 0: only keys at positions >= floor(p / chunk) * chunk are seen.  out_f32 = 1: `out` is fp32 for every dtype (its row
- * stride counts floats; no turned values then). */
+ * stride counts floats; no turned values then).  slopes (fp32 [num_heads], or NULL): s_j <- s_j - slopes[h] * (p - j) after scale
+ * and cap.  keep_first > 0 (with a window, without chunks): positions 0 .. keep_first - 1 stay visible.  gate_per_head = 1: gate
+ * is [T, num_heads].  shared_kv = 1: the values are the un-normed keys (dk = dv, no rotation); a cache row (written by
+ * shared_kv_store) is [1 / rms of every key head, fp32, 2 num_kv_heads elements rounded up to 8 | keys as projected, num_kv_heads *
+ * dk elements rounded up to 8] and s_j uses key / rms(key); a key norm's weight is folded into qnorm_w by the caller. */
+int sllm_shared_kv_store(const void* k, int64_t k_row_stride, const void* tok_seq, const void* tok_pos, const void* block_table,
+                         int max_blocks_per_seq, void* cache, int n_slots, int slot, int block_size, int64_t num_tokens,
+                         int num_kv_heads, int dk, float eps, sllm_dtype_t dtype, sllm_stream_t stream);
 int sllm_window_attention_set_simt(int on);
 int sllm_window_attention(const void* q, int64_t q_stride_t, const void* cosb, const void* sinb, const void* gate,
                           int64_t gate_stride_t, const void* cache, int n_slots, int slot, int block_size,
@@ -310,7 +318,8 @@ int sllm_window_attention(const void* q, int64_t q_stride_t, const void* cosb, c
                           int64_t out_stride_t, int64_t num_tokens, int64_t num_prefill_tokens, int num_heads, int num_kv_heads,
                           int dk, int dv, int rot_dims, int window, float scale, int sink, int pair_halves, float qk_norm_eps,
                           float softcap, const void* vcos, const void* vsin, float out_scale, const void* qnorm_w,
-                          float prenorm_eps, int chunk, int vshare, int out_f32, sllm_dtype_t dtype, sllm_stream_t stream);
+                          float prenorm_eps, int chunk, int vshare, int out_f32, const void* slopes, int keep_first,
+                          int gate_per_head, int shared_kv, sllm_dtype_t dtype, sllm_stream_t stream);
 /* diff_combine: a fp32 [T, num_kv_heads, 2, num_heads / num_kv_heads, dv] - the outputs of two score maps per head over the same
  * values (window_attention with vshare = 2, 2 * num_heads queries ordered [key/value head][map][head of the group], out_f32).
  * out[t, h] = o / sqrt(mean(o^2) + eps) * factor * sigmoid(gate[t, h]) with o = a[map 0] - lambda * a[map 1]; gate logits
@@ -320,20 +329,26 @@ int sllm_diff_combine(const void* a, const void* gate, int64_t gate_stride_t, vo
                       sllm_stream_t stream);
 
 /* ---- Sequential blocks on an fp32 residual stream whose sublayer OUTPUTS are normalised (new, stream_ops.cu).
- * embed_pair_hash: x[t] (fp32) = embed[tokens[t]] + pairs[row], row = (previous * mul_prev + token * mul_cur) mod buckets with
+ * embed_pair_hash: x[t] (fp32) = embed[tokens[t]] * scale + pairs[row], row = (previous * mul_prev + token * mul_cur) mod buckets with
  * `previous` the token one position earlier (the row above, or last_token[tok_seq[t]] (int32 per sequence row) when the step
  * starts there); a token at position 0 takes row `buckets`.  pairs may be NULL (no pair table).  x_copy (fp32, may be NULL)
  * gets the same values; h gets their rounding to dtype.  store_last_tokens then records every segment's last token. */
 int sllm_embed_pair_hash(const void* tokens, const void* tok_seq, const void* tok_pos, const void* last_token, const void* embed,
-                         const void* pairs, int buckets, int64_t mul_prev, int64_t mul_cur, void* x, void* x_copy, void* h,
-                         int64_t num_tokens, int width, sllm_dtype_t dtype, sllm_stream_t stream);
+                         const void* pairs, int buckets, int64_t mul_prev, int64_t mul_cur, float scale, void* x, void* x_copy,
+                         void* h, int64_t num_tokens, int width, sllm_dtype_t dtype, sllm_stream_t stream);
 int sllm_store_last_tokens(const void* tokens, const void* seg_starts, const void* seq_ids, void* last_token, int num_segs,
                            sllm_stream_t stream);
-/* postnorm_add_mix: X = x + gain[0] * y / sqrt(mean(y^2) + eps) per row (X = x when y is NULL); history (fp32
+/* postnorm_add_mix: X = x + gain * y / sqrt(mean(y^2) + eps) per row (X = x when y is NULL; gain: ONE number, or [width] with
+ * gain_per_channel = 1); history (fp32
  * [slots, T, width], may be NULL) slot `slot` <- X; with mix (fp32 [slot + 1], may be NULL) x <- sum_j mix[j] * history[j], else
  * x <- X; h <- x rounded to dtype.  x fp32 [T, width] in place, y dtype, gain fp32 on the device. */
-int sllm_postnorm_add_mix(void* x, const void* y, const void* gain, float eps, void* history, int slot, const void* mix, void* h,
-                          int64_t num_tokens, int width, sllm_dtype_t dtype, sllm_stream_t stream);
+int sllm_postnorm_add_mix(void* x, const void* y, const void* gain, int gain_per_channel, float eps, void* history, int slot,
+                          const void* mix, void* h, int64_t num_tokens, int width, sllm_dtype_t dtype, sllm_stream_t stream);
+/* silu_glu: u [T, 2 ff] = [gate | up] -> y [T, ff] = silu(gate) * up.  sigmoid_gate_inplace: x [T, n] *= sigmoid(gate [T, n])
+ * (gate's row stride in elements). */
+int sllm_silu_glu(const void* u, void* y, int64_t num_tokens, int ff, sllm_dtype_t dtype, sllm_stream_t stream);
+int sllm_sigmoid_gate_inplace(void* x, const void* gate, int64_t gate_stride, int64_t num_tokens, int n, sllm_dtype_t dtype,
+                              sllm_stream_t stream);
 int sllm_tanh_cap_inplace(void* x, int64_t n, float cap, sllm_dtype_t dtype, sllm_stream_t stream);
 /* moe_route_sigmoid: logits fp32 [T, experts] -> weights fp32 [T, experts]: s = sigmoid(logits); the `top` experts with the
  * largest s + bias (fp32 [experts] or NULL) get weight s, the others 0.  moe_silu_glu_scale: u [T, experts * 2 * ff] (per expert
@@ -367,6 +382,18 @@ int sllm_linear_attention(const void* q, int64_t q_stride, const void* k, int64_
                           void* out, int num_segs, int num_heads, int dk, int dv, sllm_dtype_t dtype, sllm_stream_t stream);
 int sllm_gated_rmsnorm(const void* x, const void* weight, const void* gate, int64_t gate_stride, float eps, float out_scale,
                        void* out, int64_t out_stride, int64_t num_tokens, int n, sllm_dtype_t dtype, sllm_stream_t stream);
+
+/* ---- Gated linear attention with per-sequence state (new, gla.cu); segments as for the recurrent mixers above.  Per head, with
+ * alpha[t, d] = sigmoid(z[t, d] + bias[d])^inv_tau:  S <- diag(alpha) S + k v^T (dk x dv),  o = S^T (q * q_scale),
+ * out[t] = o / sqrt(mean(o^2) + eps) * norm_w * silu(gate[t]).  q, k [T, heads * dk], v, gate, out [T, heads * dv] (dtype), z fp32
+ * [T, heads * dk] (row strides in elements), bias fp32 [heads * dk], norm_w fp32 [dv], state fp32 [rows, heads, dk, dv],
+ * o_workspace fp32 [T, heads * dv].  The first num_prefill_segs segments (num_prefill_tokens rows) are prompt portions, the rest
+ * single decoded tokens: a hint for the launch shape, any split gives the same result up to rounding.  dk <= 512. */
+int sllm_gla(const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t v_stride, const void* z,
+             int64_t z_stride, const void* bias, float inv_tau, float q_scale, const void* norm_w, float eps, const void* gate,
+             int64_t gate_stride, void* state, const void* seg_starts, const void* seq_ids, const void* tok_pos, void* o_workspace,
+             void* out, int64_t out_stride, int64_t num_tokens, int64_t num_prefill_tokens, int num_segs, int num_prefill_segs,
+             int num_heads, int dk, int dv, sllm_dtype_t dtype, sllm_stream_t stream);
 
 /* ---- Sandwich blocks: x <- x + mult * norm_b(sublayer(norm_a(x))) with RMS norms over `groups` equal consecutive parts of a row
  * (new, sandwich_ops.cu).  group_norm_add_norm: with y (dtype [T, width]) x (fp32, in place) += mult * y / rms_g(y) * wb; with

@@ -54,12 +54,13 @@ SIGNATURES = {
     "sllm_latent_kv_store": (_I, [_P, _L, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _L, _I, _I, _I, _F, _I, _P]),
     "sllm_latent_attention_set_simt": (_I, [_I]),
     "sllm_latent_attention": (_I, [_P, _L, _L, _P, _L, _L, _P, _P, _P, _L, _P, _I, _I, _I, _P, _I, _P, _P, _P, _L, _L, _L, _I, _I,
-                                   _I, _I, _I, _F, _I, _P, _I, _P]),
+                                   _I, _I, _I, _F, _P, _I, _P, _I, _P]),
     "sllm_window_kv_store": (_I, [_P, _L, _P, _L, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _L, _I, _I, _I, _I, _I, _F, _P, _P, _P, _F,
                                   _I, _I, _P]),
     "sllm_window_attention_set_simt": (_I, [_I]),
     "sllm_window_attention": (_I, [_P, _L, _P, _P, _P, _L, _P, _I, _I, _I, _P, _I, _P, _P, _P, _L, _L, _L, _I, _I, _I, _I, _I, _I,
-                                   _F, _I, _I, _F, _F, _P, _P, _F, _P, _F, _I, _I, _I, _I, _P]),
+                                   _F, _I, _I, _F, _F, _P, _P, _F, _P, _F, _I, _I, _I, _P, _I, _I, _I, _I, _P]),
+    "sllm_shared_kv_store": (_I, [_P, _L, _P, _P, _P, _I, _P, _I, _I, _I, _L, _I, _I, _F, _I, _P]),
     "sllm_diff_combine": (_I, [_P, _P, _L, _P, _L, _L, _I, _I, _I, _F, _F, _F, _I, _P]),
     "sllm_group_norm_add_norm": (_I, [_P, _P, _P, _F, _P, _P, _F, _L, _I, _I, _I, _P]),
     "sllm_group_norm_cast": (_I, [_P, _P, _P, _F, _L, _I, _I, _I, _P]),
@@ -70,9 +71,13 @@ SIGNATURES = {
     "sllm_conv_tail_update": (_I, [_P, _L, _P, _P, _P, _P, _I, _I, _I, _I, _P]),
     "sllm_mingru_scan": (_I, [_P, _L, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P]),
     "sllm_selective_scan": (_I, [_P, _L, _P, _L, _I, _P, _P, _P, _L, _I, _I, _P, _P, _L, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P]),
-    "sllm_embed_pair_hash": (_I, [_P, _P, _P, _P, _P, _P, _I, _L, _L, _P, _P, _P, _L, _I, _I, _P]),
+    "sllm_embed_pair_hash": (_I, [_P, _P, _P, _P, _P, _P, _I, _L, _L, _F, _P, _P, _P, _L, _I, _I, _P]),
     "sllm_store_last_tokens": (_I, [_P, _P, _P, _P, _I, _P]),
-    "sllm_postnorm_add_mix": (_I, [_P, _P, _P, _F, _P, _I, _P, _P, _L, _I, _I, _P]),
+    "sllm_silu_glu": (_I, [_P, _P, _L, _I, _I, _P]),
+    "sllm_sigmoid_gate_inplace": (_I, [_P, _P, _L, _L, _I, _I, _P]),
+    "sllm_gla": (_I, [_P, _L, _P, _L, _P, _L, _P, _L, _P, _F, _F, _P, _F, _P, _L, _P, _P, _P, _P, _P, _P, _L, _L, _L, _I, _I, _I, _I,
+                      _I, _I, _P]),
+    "sllm_postnorm_add_mix": (_I, [_P, _P, _P, _I, _F, _P, _I, _P, _P, _L, _I, _I, _P]),
     "sllm_tanh_cap_inplace": (_I, [_P, _L, _F, _I, _P]),
     "sllm_moe_route_sigmoid": (_I, [_P, _P, _P, _L, _I, _I, _P]),
     "sllm_moe_silu_glu_scale": (_I, [_P, _P, _P, _L, _I, _I, _I, _P]),

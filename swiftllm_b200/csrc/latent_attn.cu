@@ -5,7 +5,8 @@
 //     score(i, j) = (q_lat[i,h] . c[j] + rope(q_rot[i,h]) . k_rot[j]) * scale,   out_lat[i,h] = sum_j softmax_j(score) c[j].
 // Every token of the step is a query with its own (block-table row, position): prompt portions and single decoded tokens go
 // through the same kernel, so the result for a position does not depend on how its sequence was cut into steps.  A query at
-// position p attends to the positions max(0, p - window + 1) .. p (window <= 0: all of 0 .. p).
+// position p attends to the positions max(0, p - window + 1) .. p (window <= 0: all of 0 .. p).  With `sink` (fp32 [H]) the softmax's
+// denominator also contains exp(sink[h]): a key of that score without a value, which enters the running (maximum, sum) first.
 // Softmax, the norm of the latent and the rotation run in fp32 for every storage type.
 #include "mma_helpers.cuh"
 #include "typed_io.cuh"
@@ -60,7 +61,7 @@ __global__ void __launch_bounds__(LA_MAX_HPB * 32) latent_attn_kernel(
     const T* __restrict__ cache, int n_slots, int slot, int block_size,
     const int* __restrict__ block_table, int max_blocks_per_seq, const int* __restrict__ tok_seq,
     const int* __restrict__ tok_pos, T* __restrict__ out, int64_t out_stride_t, int64_t out_stride_h,
-    int H, int r, int dr, int rot_dims, int window, float scale) {
+    int H, int r, int dr, int rot_dims, int window, float scale, const float* __restrict__ sink) {
     extern __shared__ float smem[];
     const int D = r + dr, DP = D + 1;
     const int hpb = blockDim.x >> 5;
@@ -94,6 +95,7 @@ __global__ void __launch_bounds__(LA_MAX_HPB * 32) latent_attn_kernel(
     }
 
     float m = -INFINITY, l = 0.f;
+    if (sink != nullptr && live) { m = sink[h]; l = 1.f; }
     float acc[KR];
 #pragma unroll
     for (int k = 0; k < KR; k++) acc[k] = 0.f;
@@ -164,7 +166,7 @@ __global__ void __launch_bounds__(LM_NW * 32) latent_attn_mma_kernel(
     int64_t gate_stride_t, const T* __restrict__ cache, int n_slots, int slot, int block_size,
     const int* __restrict__ block_table, int max_blocks_per_seq, const int* __restrict__ tok_seq,
     const int* __restrict__ tok_pos, T* __restrict__ out, int64_t out_stride_t, int64_t out_stride_h, int H, int r, int dr,
-    int rot_dims, int window, float scale, int nsplit, float* __restrict__ partial) {
+    int rot_dims, int window, float scale, int nsplit, float* __restrict__ partial, const float* __restrict__ sink) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int D = r + dr, LD = D + 8, LP = LM_KT + 8, LS = LM_KT + 1;
     T* Qs = reinterpret_cast<T*>(smem_raw);                 // [16][LD]
@@ -205,7 +207,11 @@ __global__ void __launch_bounds__(LM_NW * 32) latent_attn_mma_kernel(
             for (int d = lane; d < D; d += 32) stf(qw + d, 0.f);
         }
     }
-    if (threadIdx.x < 16) { ms[threadIdx.x] = -INFINITY; ls[threadIdx.x] = 0.f; }
+    if (threadIdx.x < 16) {
+        const bool s0 = sink != nullptr && blockIdx.z == 0 && h0 + (int)threadIdx.x < H;      // the sink counts in ONE key split
+        ms[threadIdx.x] = s0 ? sink[h0 + threadIdx.x] : -INFINITY;
+        ls[threadIdx.x] = s0 ? 1.f : 0.f;
+    }
 
     float acc[NT][4];
 #pragma unroll
@@ -370,7 +376,7 @@ static int launch_latent_attn_mma(const void* q_lat, int64_t ql_st, int64_t ql_s
                                   int n_slots, int slot, int block_size, const void* block_table, int max_blocks_per_seq,
                                   const void* tok_seq, const void* tok_pos, void* out, int64_t out_st, int64_t out_sh,
                                   int64_t num_tokens, int H, int r, int dr, int rot_dims, int window, float scale,
-                                  cudaStream_t stream, int nsplit, void* partial) {
+                                  const void* sink, cudaStream_t stream, int nsplit, void* partial) {
     const int D = r + dr;
     const size_t smem = ((size_t)(16 + LM_KT) * (D + 8) + 16 * (LM_KT + 8)) * 2 + (16 * (LM_KT + 1) + 48) * sizeof(float);
     SLLM_REQUIRE(smem <= 200 * 1024, "latent_attention: r + dr = %d needs %zu bytes of shared memory", D, smem);
@@ -384,7 +390,8 @@ static int launch_latent_attn_mma(const void* q_lat, int64_t ql_st, int64_t ql_s
     kern<<<grid, LM_NW * 32, smem, stream>>>(
         (const T*)q_lat, ql_st, ql_sh, (const T*)q_rot, qr_st, qr_sh, (const float*)cosb, (const float*)sinb, (const T*)gate,
         gate_st, (const T*)cache, n_slots, slot, block_size, (const int*)block_table, max_blocks_per_seq, (const int*)tok_seq,
-        (const int*)tok_pos, (T*)out, out_st, out_sh, H, r, dr, rot_dims, window, scale, nsplit, (float*)partial);
+        (const int*)tok_pos, (T*)out, out_st, out_sh, H, r, dr, rot_dims, window, scale, nsplit, (float*)partial,
+        (const float*)sink);
     if (int rc = check_launch("latent_attention (mma)")) return rc;
     if (nsplit > 1) {
         latent_attn_combine_kernel<T><<<(unsigned)cdiv(num_tokens * H, 4), 128, 0, stream>>>(
@@ -412,7 +419,7 @@ static int launch_latent_attn(const void* q_lat, int64_t ql_st, int64_t ql_sh, c
                               int n_slots, int slot, int block_size, const void* block_table, int max_blocks_per_seq,
                               const void* tok_seq, const void* tok_pos, void* out, int64_t out_st, int64_t out_sh,
                               int64_t num_tokens, int H, int r, int dr, int rot_dims, int window, float scale,
-                              cudaStream_t stream) {
+                              const void* sink, cudaStream_t stream) {
     const int hpb = H < LA_MAX_HPB ? H : LA_MAX_HPB;
     const int D = r + dr;
     const size_t smem = ((size_t)hpb * D + (size_t)LA_TILE * (D + 1)) * sizeof(float);
@@ -427,7 +434,7 @@ static int launch_latent_attn(const void* q_lat, int64_t ql_st, int64_t ql_sh, c
     kern<<<grid, hpb * 32, smem, stream>>>(
         (const T*)q_lat, ql_st, ql_sh, (const T*)q_rot, qr_st, qr_sh, (const float*)cosb, (const float*)sinb, (const T*)gate,
         gate_st, (const T*)cache, n_slots, slot, block_size, (const int*)block_table, max_blocks_per_seq, (const int*)tok_seq,
-        (const int*)tok_pos, (T*)out, out_st, out_sh, H, r, dr, rot_dims, window, scale);
+        (const int*)tok_pos, (T*)out, out_st, out_sh, H, r, dr, rot_dims, window, scale, (const float*)sink);
     return check_launch("latent_attention");
 }
 
@@ -469,7 +476,7 @@ int sllm_latent_attention(const void* q_lat, int64_t q_lat_stride_t, int64_t q_l
                           const void* gate, int64_t gate_stride_t, const void* cache, int n_slots, int slot, int block_size,
                           const void* block_table, int max_blocks_per_seq, const void* tok_seq, const void* tok_pos,
                           void* out, int64_t out_stride_t, int64_t out_stride_h, int64_t num_tokens, int num_heads, int r,
-                          int dr, int rot_dims, int window, float scale, int num_splits, void* split_workspace,
+                          int dr, int rot_dims, int window, float scale, const void* sink, int num_splits, void* split_workspace,
                           sllm_dtype_t dtype, sllm_stream_t stream) {
     SLLM_REQUIRE(num_tokens >= 0 && num_heads > 0 && r > 0 && r <= 1024 && dr >= 0 && rot_dims >= 0 && rot_dims <= dr &&
                  rot_dims % 2 == 0, "latent_attention: bad shape (heads %d, r %d <= 1024, dr %d, rot_dims %d)", num_heads, r, dr,
@@ -481,7 +488,7 @@ int sllm_latent_attention(const void* q_lat, int64_t q_lat_stride_t, int64_t q_l
                  (rot_dims == 0 || (cosb && sinb)), "latent_attention: null pointer");
 #define SLLM_LA_ARGS q_lat, q_lat_stride_t, q_lat_stride_h, q_rot, q_rot_stride_t, q_rot_stride_h, cosb, sinb, gate,            \
                      gate_stride_t, cache, n_slots, slot, block_size, block_table, max_blocks_per_seq, tok_seq, tok_pos, out,   \
-                     out_stride_t, out_stride_h, num_tokens, num_heads, r, dr, rot_dims, window, scale, (cudaStream_t)stream
+                     out_stride_t, out_stride_h, num_tokens, num_heads, r, dr, rot_dims, window, scale, sink, (cudaStream_t)stream
     // 16-bit storage and 16-element-aligned rows: tensor cores; everything else: the fp32 CUDA-core kernel
     const size_t mma_smem = ((size_t)(16 + LM_KT) * (r + dr + 8) + 16 * (LM_KT + 8)) * 2 + (16 * (LM_KT + 1) + 48) * sizeof(float);
     const bool mma = dtype != SLLM_F32 && r % 16 == 0 && dr % 16 == 0 && mma_smem <= 200 * 1024 && !sllm_latent_attention_force_simt;

@@ -20,6 +20,12 @@
 //   vshare > 1         `vshare` neighbouring key heads share ONE value head (value head = key head / vshare; the cache row holds
 //                      G keys and G / vshare values): several score maps over the same values, each its own query head
 //   out_f32            the output is written as fp32 whatever the storage type (a combine step follows)
+//   slopes             a bias on the distance: score <- score - slopes[h] * (i - j) after the scale (and cap)
+//   keep_first > 0     with a window: the sequence's first keep_first positions stay visible (at their true positions)
+//   gate_per_head      ONE gate logit per query head ([T, H]) instead of one per output entry
+//   shared_kv          the values are the un-normed keys: the cache row is [ inv (G fp32 values in 2 G elements, rounded up to 8) |
+//                      k (G x dk as projected, rounded up to 8) ], inv = 1 / sqrt(mean(k^2) + eps) of the head; the norm's weight
+//                      belongs to the query weights (q . (inv k w) = inv (q w) . k), so ONE staged tile serves as K and V
 // diff_combine: per token and head, o = a1 - lambda * a2 of two maps' outputs, o / sqrt(mean(o^2) + eps) * factor * sigmoid(gate).
 #include "mma_helpers.cuh"
 #include "typed_io.cuh"
@@ -46,6 +52,14 @@ __device__ __forceinline__ float rot_entry(const T* __restrict__ x, int j, int r
     const float a = pre_entry(x, 2 * i, inv, nw), b = pre_entry(x, 2 * i + 1, inv, nw);
     return (j & 1) ? b * cs[i] + a * sn[i] : a * cs[i] - b * sn[i];
 }
+
+// the shared_kv cache row: first element of the keys, elements per row
+__host__ __device__ __forceinline__ int shared_kv_key_offset(int G) { return (2 * G + 7) / 8 * 8; }
+__host__ __device__ __forceinline__ int shared_kv_row(int G, int dk) { return shared_kv_key_offset(G) + (G * dk + 7) / 8 * 8; }
+
+// What a query at position p sees, walked as ONE list of keys: entries 0 .. nk - 1 are the kept first positions that lie before the
+// window's start `lo`, the rest are lo, lo + 1, ..
+__device__ __forceinline__ int key_position(int v, int nk, int lo) { return v < nk ? v : v - nk + lo; }
 
 // ------------------------------------------------------------------ cache store
 // One CTA per token, one warp per key/value head at a time: rotate k (and divide it by its root mean square), rotate or copy v,
@@ -95,6 +109,33 @@ __global__ void __launch_bounds__(128) window_kv_store_kernel(
     }
 }
 
+// One CTA per token, one warp per key head at a time: the row of the shared_kv layout (see the top of the file).
+template <typename T>
+__global__ void __launch_bounds__(128) shared_kv_store_kernel(
+    const T* __restrict__ k, int64_t k_stride, const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
+    const int* __restrict__ block_table, int max_blocks_per_seq, T* __restrict__ cache, int n_slots, int slot, int block_size,
+    int G, int dk, float eps) {
+    const int64_t t = blockIdx.x;
+    const int pos = tok_pos[t];
+    const int blk = block_table[(int64_t)tok_seq[t] * max_blocks_per_seq + pos / block_size];
+    const int koff = shared_kv_key_offset(G);
+    T* dst = cache + (((int64_t)blk * n_slots + slot) * block_size + pos % block_size) * shared_kv_row(G, dk);
+    float* inv = reinterpret_cast<float*>(dst);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
+    for (int g = warp; g < G; g += nwarps) {
+        const T* x = k + t * k_stride + g * dk;
+        float ss = 0.f;
+        for (int j = lane; j < dk; j += 32) {
+            const T v = x[j];
+            const float f = ldf(&v);
+            ss += f * f;
+            dst[koff + g * dk + j] = v;
+        }
+        ss = warp_sum(ss);
+        if (lane == 0) inv[g] = 1.f / sqrtf(ss / (float)dk + eps);
+    }
+}
+
 // ------------------------------------------------------------------ attention (fp32 CUDA cores)
 constexpr int WA_TILE = 32;        // keys per tile: one per lane in the score phase
 constexpr int WA_MAX_HPB = 8;      // query heads (warps) per CTA: heads of ONE key/value group, they share the staged tile
@@ -110,7 +151,8 @@ __global__ void __launch_bounds__(WA_MAX_HPB * 32) window_attn_kernel(
     const int* __restrict__ tok_pos, T* __restrict__ out, int64_t out_stride_t,  // [T, H, dv]
     int H, int G, int dk, int dv, int rot_dims, int window, float scale, float sink, int halves, float qk_norm_eps,
     float softcap, const float* __restrict__ vcos, const float* __restrict__ vsin, float out_scale,
-    const float* __restrict__ qnorm_w, float prenorm_eps, int chunk, int vshare, int out_f32) {
+    const float* __restrict__ qnorm_w, float prenorm_eps, int chunk, int vshare, int out_f32, const float* __restrict__ slopes,
+    int keep_first, int gate_per_head, int shared_kv) {
     extern __shared__ float smem[];
     const int KP = dk + 1;
     const int hpb = blockDim.x >> 5;
@@ -118,13 +160,16 @@ __global__ void __launch_bounds__(WA_MAX_HPB * 32) window_attn_kernel(
     float* kt = qs + hpb * dk;                 // [WA_TILE][dk + 1]
     float* vt = kt + WA_TILE * KP;             // [WA_TILE][dv]
     float* os = vt + WA_TILE * dv;             // [hpb][dv]: the head's output before it is turned back (vcos only)
+    float* kinv = os + hpb * dv;               // [WA_TILE]: the keys' 1 / rms (shared_kv only)
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int64_t t = blockIdx.x;
     const int h = blockIdx.y * hpb + warp;
     const int g = (blockIdx.y * hpb) / (H / G);
     const int pos = tok_pos[t];
     const int* bt = block_table + (int64_t)tok_seq[t] * max_blocks_per_seq;
-    const int row = G * dk + (G / vshare) * dv;
+    const int row = shared_kv ? shared_kv_row(G, dk) : G * dk + (G / vshare) * dv;
+    const int koff = shared_kv ? shared_kv_key_offset(G) : 0;
+    const float slope = slopes != nullptr ? slopes[h] : 0.f;
 
     {
         float* qw = qs + warp * dk;
@@ -155,15 +200,23 @@ __global__ void __launch_bounds__(WA_MAX_HPB * 32) window_attn_kernel(
 
     int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
     if (chunk > 0) lo = max(lo, pos / chunk * chunk);
-    for (int base = lo; base <= pos; base += WA_TILE) {
+    const int nk = window > 0 ? min(keep_first, lo) : 0;
+    const int total = nk + pos - lo + 1;
+    const float* vbase = shared_kv ? kt : vt;
+    const int VP = shared_kv ? KP : dv;
+    for (int base = 0; base < total; base += WA_TILE) {
         __syncthreads();                       // the previous tile is no longer read (and qs is written, first time round)
-        const int nkeys = min(WA_TILE, pos - base + 1);
+        const int nkeys = min(WA_TILE, total - base);
         for (int jj = warp; jj < nkeys; jj += hpb) {
-            const int kp = base + jj;
+            const int kp = key_position(base + jj, nk, lo);
             const T* src = cache + (((int64_t)bt[kp / block_size] * n_slots + slot) * block_size + kp % block_size) * row;
-            const T* ks = src + g * dk;
-            const T* vs = src + G * dk + (g / vshare) * dv;
+            const T* ks = src + koff + g * dk;
             for (int d = lane; d < dk; d += 32) kt[jj * KP + d] = ldf(ks + d);
+            if (shared_kv) {
+                if (lane == 0) kinv[jj] = reinterpret_cast<const float*>(src)[g];
+                continue;
+            }
+            const T* vs = src + G * dk + (g / vshare) * dv;
             for (int d = lane; d < dv; d += 32) vt[jj * dv + d] = ldf(vs + d);
         }
         __syncthreads();
@@ -173,9 +226,11 @@ __global__ void __launch_bounds__(WA_MAX_HPB * 32) window_attn_kernel(
             const float* kr = kt + lane * KP;
             float a = 0.f;
             for (int d = 0; d < dk; d++) a += qw[d] * kr[d];
+            if (shared_kv) a *= kinv[lane];
             s = softcap > 0.f ? softcap * tanhf(a / softcap) : a;
+            s -= slope * (float)(pos - key_position(base + lane, nk, lo));
         }
-        const float m_new = fmaxf(m, warp_max(s));          // finite: key `base` is always visible
+        const float m_new = fmaxf(m, warp_max(s));          // finite: every tile has a visible key
         const float alpha = expf(m - m_new);                // 0 on the first tile without a sink (m = -inf)
         const float p = lane < nkeys ? expf(s - m_new) : 0.f;
         l = l * alpha + warp_sum(p);
@@ -183,7 +238,7 @@ __global__ void __launch_bounds__(WA_MAX_HPB * 32) window_attn_kernel(
         for (int k = 0; k < KR; k++) acc[k] *= alpha;
         for (int jj = 0; jj < nkeys; jj++) {
             const float pj = __shfl_sync(0xffffffffu, p, jj);
-            const float* vr = vt + jj * dv;
+            const float* vr = vbase + jj * VP;
 #pragma unroll
             for (int k = 0; k < KR; k++) {
                 const int d = lane + 32 * k;
@@ -194,7 +249,8 @@ __global__ void __launch_bounds__(WA_MAX_HPB * 32) window_attn_kernel(
     }
     float denom = l;
     T* o = out + t * out_stride_t + (int64_t)h * dv;
-    const T* gr = gate != nullptr ? gate + t * gate_stride_t + (int64_t)h * dv : nullptr;
+    const T* gr = gate != nullptr && !gate_per_head ? gate + t * gate_stride_t + (int64_t)h * dv : nullptr;
+    if (gate != nullptr && gate_per_head) out_scale *= 1.f / (1.f + expf(-ldf(gate + t * gate_stride_t + h)));
     if (vcos != nullptr) {
         // the sum of turned values is turned back by the query's own position: pair (a, b) -> (a c + b s, b c - a s)
         float* ow = os + warp * dv;
@@ -253,18 +309,21 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
     const int* __restrict__ tok_pos, T* __restrict__ out, int64_t out_stride_t, int row0, int nrows, int qt, int hq, int hqp_log2,
     int H, int G, int dk, int dv, int rot_dims, int window, float scale_log2, float sink, int halves, float qk_norm_eps,
     float softcap, const float* __restrict__ vcos, const float* __restrict__ vsin, float out_scale,
-    const float* __restrict__ qnorm_w, float prenorm_eps, int chunk, int vshare, int out_f32) {
+    const float* __restrict__ qnorm_w, float prenorm_eps, int chunk, int vshare, int out_f32, const float* __restrict__ slopes,
+    int keep_first, int gate_per_head, int shared_kv) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int PQ = dk * 2 + 16, PK = dk * 2 + 16, PV = dv * 2 + 16;            // row pitches in bytes
     unsigned char* Qs = smem_raw;                                              // [64][PQ]
     unsigned char* Ks = Qs + WT_ROWS * PQ;                                     // [2][64][PK]
-    unsigned char* Vs = Ks + 2 * WT_KEYS * PK;                                 // [2][64][PV]
+    unsigned char* Vs = shared_kv ? Ks : Ks + 2 * WT_KEYS * PK;                // [2][64][PV] (shared_kv: the key tile itself)
+    float* kinv = reinterpret_cast<float*>(Ks + 2 * WT_KEYS * PK);             // [2][64]: the keys' 1 / rms (shared_kv only)
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int g = blockIdx.y;
     const int hqp = 1 << hqp_log2;
     const int t_first = row0 + blockIdx.x * qt;
     const int ntok = min(qt, row0 + nrows - t_first);
-    const int row_elems = G * dk + (G / vshare) * dv;
+    const int row_elems = shared_kv ? shared_kv_row(G, dk) : G * dk + (G / vshare) * dv;
+    const int koff = shared_kv ? shared_kv_key_offset(G) : 0;
     const int ck = dk >> 3, cv = dv >> 3;                                      // 16-byte chunks per key / value row
     const int half = rot_dims >> 1;
     // with a score cap: cap * tanh(s * scale / cap), then to base 2
@@ -281,27 +340,33 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
         int lo = (window > 0 && pos0 - window + 1 > 0) ? pos0 - window + 1 : 0;
         if (chunk > 0) lo = max(lo, pos0 / chunk * chunk);
         const int hi = pos0 + n - 1;
-        const int ntiles = (hi - lo) / WT_KEYS + 1;
+        const int nk = window > 0 ? min(keep_first, lo) : 0;
+        const int total = nk + hi - lo + 1;                                    // keys the segment's rows see together
+        const int ntiles = (total - 1) / WT_KEYS + 1;
         __syncthreads();                                                       // the previous segment's tiles and queries are done with
 
         // two threads per key row, alternating 16-byte chunks: ONE block-table lookup and address per thread and tile
         auto load_tile = [&](int it) {
             constexpr int TPR = 128 / WT_KEYS;                                 // threads per key row
             const int st = it & 1, jj = tid / TPR, part = tid % TPR;
-            const int kp = lo + it * WT_KEYS + jj;
+            const int kp = key_position(it * WT_KEYS + jj, nk, lo);
             const bool ok = kp <= hi;
             const T* krow = cache;
             const T* vrow = cache;
             if (ok) {
                 const int b = kp / block_size;
                 const int64_t rowi = ((int64_t)bt[b] * n_slots + slot) * block_size + (kp - b * block_size);
-                krow = cache + rowi * row_elems + g * dk;
+                krow = cache + rowi * row_elems + koff + g * dk;
                 vrow = cache + rowi * row_elems + G * dk + (g / vshare) * dv;
+                if (shared_kv && part == 0) cp_async4(smem_u32(kinv + st * WT_KEYS + jj), cache + rowi * row_elems + 2 * g);
+            } else if (shared_kv && part == 0) {
+                kinv[st * WT_KEYS + jj] = 0.f;
             }
             const int nb = ok ? 16 : 0;
             const uint32_t kd = smem_u32(Ks + (st * WT_KEYS + jj) * PK), vd = smem_u32(Vs + (st * WT_KEYS + jj) * PV);
             for (int ch = part; ch < ck; ch += TPR) cp_async16(kd + ch * 16, ok ? krow + ch * 8 : krow, nb);
-            for (int ch = part; ch < cv; ch += TPR) cp_async16(vd + ch * 16, ok ? vrow + ch * 8 : vrow, nb);
+            if (!shared_kv)
+                for (int ch = part; ch < cv; ch += TPR) cp_async16(vd + ch * 16, ok ? vrow + ch * 8 : vrow, nb);
             cp_async_commit();
         };
         load_tile(0);
@@ -362,6 +427,8 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
         int w_lo = window > 0 ? max(0, pos0 + wj_min - window + 1) : 0;
         if (chunk > 0) w_lo = max(w_lo, (pos0 + wj_min) / chunk * chunk);
         const int w_hi = pos0 + wj_max;
+        const float sl_a = slopes != nullptr && live_a ? slopes[g * hq + (r_a & (hqp - 1))] * 1.4426950408889634f : 0.f;
+        const float sl_b = slopes != nullptr && live_b ? slopes[g * hq + (r_b & (hqp - 1))] * 1.4426950408889634f : 0.f;
         float m_a = sink > 0.f ? 0.f : -INFINITY, m_b = m_a;
         float l_a = (lane & 3) == 0 ? sink : 0.f, l_b = l_a;
         float o[DMAX / 8][4];
@@ -371,8 +438,9 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
         for (int it = 0; it < ntiles; it++) {
             if (it + 1 < ntiles) { load_tile(it + 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
             __syncthreads();                                                   // tile `it` (and, first time, the queries) visible
-            const int base = lo + it * WT_KEYS;
-            if (warp_live && base <= w_hi && base + WT_KEYS - 1 >= w_lo) {
+            const int base = it * WT_KEYS;                                     // the tile's first entry in the list of visible keys
+            const int kp_first = key_position(base, nk, lo), kp_last = key_position(base + WT_KEYS - 1, nk, lo);
+            if (warp_live && kp_first <= w_hi && (kp_last >= w_lo || kp_first < keep_first)) {
                 const unsigned char* Kt = Ks + (it & 1) * WT_KEYS * PK;
                 const unsigned char* Vt = Vs + (it & 1) * WT_KEYS * PV;
                 float sc[WT_KEYS / 8][4];
@@ -394,16 +462,27 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
                         }
                     }
                 }
+                if (shared_kv) {
+                    const float* ki = kinv + (it & 1) * WT_KEYS + (lane & 3) * 2;
+#pragma unroll
+                    for (int nt = 0; nt < WT_KEYS / 8; nt++) {
+                        const float2 f = *reinterpret_cast<const float2*>(ki + nt * 8);
+                        sc[nt][0] *= f.x; sc[nt][1] *= f.y; sc[nt][2] *= f.x; sc[nt][3] *= f.y;
+                    }
+                }
                 // mask, running maximum
                 float mx_a = -INFINITY, mx_b = -INFINITY;
 #pragma unroll
                 for (int nt = 0; nt < WT_KEYS / 8; nt++) {
 #pragma unroll
                     for (int e = 0; e < 2; e++) {
-                        const int kp = base + nt * 8 + (lane & 3) * 2 + e;
-                        const bool va = live_a && kp <= pos_a && kp >= lo_a, vb = live_b && kp <= pos_b && kp >= lo_b;
-                        const float sa = softcap > 0.f ? cap_out * tanhf(sc[nt][e] * cap_in) : sc[nt][e] * scale_log2;
-                        const float sb = softcap > 0.f ? cap_out * tanhf(sc[nt][2 + e] * cap_in) : sc[nt][2 + e] * scale_log2;
+                        const int kp = key_position(base + nt * 8 + (lane & 3) * 2 + e, nk, lo);
+                        const bool kept = kp < keep_first;
+                        const bool va = live_a && kp <= pos_a && (kp >= lo_a || kept), vb = live_b && kp <= pos_b && (kp >= lo_b || kept);
+                        float sa = softcap > 0.f ? cap_out * tanhf(sc[nt][e] * cap_in) : sc[nt][e] * scale_log2;
+                        float sb = softcap > 0.f ? cap_out * tanhf(sc[nt][2 + e] * cap_in) : sc[nt][2 + e] * scale_log2;
+                        sa -= sl_a * (float)(pos_a - kp);
+                        sb -= sl_b * (float)(pos_b - kp);
                         sc[nt][e] = va ? sa : -INFINITY;
                         sc[nt][2 + e] = vb ? sb : -INFINITY;
                         mx_a = fmaxf(mx_a, sc[nt][e]);
@@ -475,9 +554,9 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
                 float ya = (a * c + b * sn) * out_scale, yb = (b * c - a * sn) * out_scale;
                 T* orow = out + t * out_stride_t + (int64_t)(g * hq + hh) * dv;
                 if (gate != nullptr) {
-                    const T* grow = gate + t * gate_stride_t + (int64_t)(g * hq + hh) * dv;
-                    ya *= 1.f / (1.f + __expf(-ldf(grow + da)));
-                    yb *= 1.f / (1.f + __expf(-ldf(grow + db)));
+                    const T* grow = gate + t * gate_stride_t + (gate_per_head ? g * hq + hh : (int64_t)(g * hq + hh) * dv);
+                    ya *= 1.f / (1.f + __expf(-ldf(grow + (gate_per_head ? 0 : da))));
+                    yb *= 1.f / (1.f + __expf(-ldf(grow + (gate_per_head ? 0 : db))));
                 }
                 stf(orow + da, ya);
                 stf(orow + db, yb);
@@ -492,9 +571,10 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
             const int r = e ? r_b : r_a;
             const int64_t t = ts + (r >> hqp_log2);
             const int h = g * hq + (r & (hqp - 1));
-            const float inv = out_scale / (e ? l_b : l_a);
+            float inv = out_scale / (e ? l_b : l_a);
+            if (gate != nullptr && gate_per_head) inv *= 1.f / (1.f + __expf(-ldf(gate + t * gate_stride_t + h)));
             T* orow = out + t * out_stride_t + (int64_t)h * dv;
-            const T* grow = gate != nullptr ? gate + t * gate_stride_t + (int64_t)h * dv : nullptr;
+            const T* grow = gate != nullptr && !gate_per_head ? gate + t * gate_stride_t + (int64_t)h * dv : nullptr;
 #pragma unroll
             for (int nt = 0; nt < DMAX / 8; nt++) {
                 const int d = nt * 8 + (lane & 3) * 2;
@@ -564,7 +644,8 @@ static int launch_window_attn_mma(const void* q, int64_t q_stride_t, const void*
                                   void* out, int64_t out_stride_t, int64_t num_tokens, int64_t num_prefill, int H, int G, int dk,
                                   int dv, int rot_dims, int window, float scale, float sink, int halves, float qk_norm_eps,
                                   float softcap, const void* vcos, const void* vsin, float out_scale, const void* qnorm_w,
-                                  float prenorm_eps, int chunk, int vshare, int out_f32, cudaStream_t stream) {
+                                  float prenorm_eps, int chunk, int vshare, int out_f32, const void* slopes, int keep_first,
+                                  int gate_per_head, int shared_kv, cudaStream_t stream) {
     static unsigned long long attr_mask = 0;
     const int hq = H / G;
     int hqp_log2 = 0;
@@ -586,14 +667,14 @@ static int launch_window_attn_mma(const void* q, int64_t q_stride_t, const void*
         // measured on B200 (128 + 128 per head): prompt portions 24 - 26 % faster with 32-key tiles (three CTAs per SM instead of
         // two); decoded tokens faster with 64-key tiles at 512 CTAs (357 vs 385 us), with 32-key tiles at 2048 CTAs (950 vs 1220 us)
         const int keys = (k == 0 || count * G >= 7 * (int64_t)num_sms) ? 32 : 64;
-        size_t smem = (size_t)WT_ROWS * (dk * 2 + 16) + 2 * (size_t)keys * ((dk * 2 + 16) + (dv * 2 + 16));
+        size_t smem = (size_t)WT_ROWS * (dk * 2 + 16) + 2 * (size_t)keys * ((dk * 2 + 16) + (shared_kv ? sizeof(float) : dv * 2 + 16));
         if (vcos != nullptr && smem < (size_t)WT_ROWS * dv * sizeof(float)) smem = (size_t)WT_ROWS * dv * sizeof(float);
         (keys == 32 ? kern_prompt : kern_decode)<<<dim3((unsigned)cdiv(count, qt), (unsigned)G), 128, smem, stream>>>(
             (const T*)q, q_stride_t, (const float*)cosb, (const float*)sinb, (const T*)gate, gate_stride_t, (const T*)cache,
             n_slots, slot, block_size, (const int*)block_table, max_blocks_per_seq, (const int*)tok_seq, (const int*)tok_pos,
             (T*)out, out_stride_t, (int)first, (int)count, qt, hq, hqp_log2, H, G, dk, dv, rot_dims, window, scale_log2, sink,
             halves, qk_norm_eps, softcap, (const float*)vcos, (const float*)vsin, out_scale, (const float*)qnorm_w, prenorm_eps,
-            chunk, vshare, out_f32);
+            chunk, vshare, out_f32, (const float*)slopes, keep_first, gate_per_head, shared_kv);
     }
     return check_launch("window_attention (tensor cores)");
 }
@@ -611,10 +692,11 @@ static int launch_window_attn(const void* q, int64_t q_stride_t, const void* cos
                               int64_t out_stride_t, int64_t num_tokens, int H, int G, int dk, int dv, int rot_dims, int window,
                               float scale, float sink, int halves, float qk_norm_eps, float softcap, const void* vcos,
                               const void* vsin, float out_scale, const void* qnorm_w, float prenorm_eps, int chunk, int vshare,
-                              int out_f32, cudaStream_t stream) {
+                              int out_f32, const void* slopes, int keep_first, int gate_per_head, int shared_kv,
+                              cudaStream_t stream) {
     static unsigned long long attr_mask = 0;
     const int hpb = heads_per_cta(H / G);
-    const size_t smem = ((size_t)hpb * dk + (size_t)WA_TILE * (dk + 1) + (size_t)WA_TILE * dv + (size_t)hpb * dv) * sizeof(float);
+    const size_t smem = ((size_t)hpb * dk + (size_t)WA_TILE * (dk + 1) + (size_t)WA_TILE * dv + (size_t)hpb * dv + WA_TILE) * sizeof(float);
     SLLM_REQUIRE(smem <= 200 * 1024, "window_attention: head sizes %d / %d need %zu bytes of shared memory", dk, dv, smem);
     auto kern = window_attn_kernel<T, KR>;
     if (first_use_on_this_device(attr_mask))
@@ -623,7 +705,8 @@ static int launch_window_attn(const void* q, int64_t q_stride_t, const void* cos
         (const T*)q, q_stride_t, (const float*)cosb, (const float*)sinb, (const T*)gate, gate_stride_t, (const T*)cache, n_slots,
         slot, block_size, (const int*)block_table, max_blocks_per_seq, (const int*)tok_seq, (const int*)tok_pos, (T*)out,
         out_stride_t, H, G, dk, dv, rot_dims, window, scale, sink, halves, qk_norm_eps, softcap, (const float*)vcos,
-        (const float*)vsin, out_scale, (const float*)qnorm_w, prenorm_eps, chunk, vshare, out_f32);
+        (const float*)vsin, out_scale, (const float*)qnorm_w, prenorm_eps, chunk, vshare, out_f32, (const float*)slopes, keep_first,
+        gate_per_head, shared_kv);
     return check_launch("window_attention");
 }
 
@@ -657,6 +740,19 @@ int sllm_window_kv_store(const void* k, int64_t k_row_stride, const void* v, int
     return check_launch("window_kv_store");
 }
 
+int sllm_shared_kv_store(const void* k, int64_t k_row_stride, const void* tok_seq, const void* tok_pos, const void* block_table,
+                         int max_blocks_per_seq, void* cache, int n_slots, int slot, int block_size, int64_t num_tokens,
+                         int num_kv_heads, int dk, float eps, sllm_dtype_t dtype, sllm_stream_t stream) {
+    SLLM_REQUIRE(num_tokens >= 0 && num_kv_heads > 0 && dk > 0, "shared_kv_store: bad shape (kv heads %d, dk %d)", num_kv_heads, dk);
+    SLLM_REQUIRE(slot >= 0 && slot < n_slots && block_size > 0, "shared_kv_store: bad cache slot %d of %d", slot, n_slots);
+    if (num_tokens == 0) return 0;
+    SLLM_REQUIRE(k && tok_seq && tok_pos && block_table && cache, "shared_kv_store: null pointer");
+    SLLM_DISPATCH_DTYPE_F32(dtype, (shared_kv_store_kernel<T><<<(unsigned)num_tokens, 128, 0, (cudaStream_t)stream>>>(
+        (const T*)k, k_row_stride, (const int*)tok_seq, (const int*)tok_pos, (const int*)block_table, max_blocks_per_seq,
+        (T*)cache, n_slots, slot, block_size, num_kv_heads, dk, eps)));
+    return check_launch("shared_kv_store");
+}
+
 int sllm_window_attention_set_simt(int on) {
     const int old = g_window_simt ? 1 : 0;
     g_window_simt = on != 0;
@@ -669,7 +765,12 @@ int sllm_window_attention(const void* q, int64_t q_stride_t, const void* cosb, c
                           int64_t out_stride_t, int64_t num_tokens, int64_t num_prefill_tokens, int num_heads, int num_kv_heads,
                           int dk, int dv, int rot_dims, int window, float scale, int sink, int pair_halves, float qk_norm_eps,
                           float softcap, const void* vcos, const void* vsin, float out_scale, const void* qnorm_w,
-                          float prenorm_eps, int chunk, int vshare, int out_f32, sllm_dtype_t dtype, sllm_stream_t stream) {
+                          float prenorm_eps, int chunk, int vshare, int out_f32, const void* slopes, int keep_first,
+                          int gate_per_head, int shared_kv, sllm_dtype_t dtype, sllm_stream_t stream) {
+    SLLM_REQUIRE(keep_first >= 0 && (keep_first == 0 || chunk == 0), "window_attention: kept first positions (%d) exclude chunks",
+                 keep_first);
+    SLLM_REQUIRE(!shared_kv || (dk == dv && vshare == 1 && rot_dims == 0 && qk_norm_eps < 0.f && vcos == nullptr),
+                 "window_attention: values that are the un-normed keys need dk = dv and no rotation (dk %d, dv %d)", dk, dv);
     SLLM_REQUIRE(vshare >= 1 && num_kv_heads % vshare == 0 && chunk >= 0 && (!out_f32 || vcos == nullptr),
                  "window_attention: %d key heads in runs of %d; chunk %d >= 0; fp32 output excludes turned values", num_kv_heads,
                  vshare, chunk);
@@ -692,7 +793,8 @@ int sllm_window_attention(const void* q, int64_t q_stride_t, const void* cosb, c
     SLLM_DISPATCH_DTYPE(dtype, return (launch_window_attn_mma<T, DMAX>(q, q_stride_t, cosb, sinb, gate, gate_stride_t, cache,  \
         n_slots, slot, block_size, block_table, max_blocks_per_seq, tok_seq, tok_pos, out, out_stride_t, num_tokens,         \
         num_prefill_tokens, num_heads, num_kv_heads, dk, dv, rot_dims, window, scale, sinkw, pair_halves, qk_norm_eps, softcap, \
-        vcos, vsin, out_scale, qnorm_w, prenorm_eps, chunk, vshare, out_f32, (cudaStream_t)stream)))
+        vcos, vsin, out_scale, qnorm_w, prenorm_eps, chunk, vshare, out_f32, slopes, keep_first, gate_per_head, shared_kv,        \
+        (cudaStream_t)stream)))
         if (dk <= 64 && dv <= 64) { WA_MMA(64); }
         else { WA_MMA(128); }
 #undef WA_MMA
@@ -701,7 +803,8 @@ int sllm_window_attention(const void* q, int64_t q_stride_t, const void* cosb, c
     SLLM_DISPATCH_DTYPE_F32(dtype, return (launch_window_attn<T, KR>(q, q_stride_t, cosb, sinb, gate, gate_stride_t, cache,   \
         n_slots, slot, block_size, block_table, max_blocks_per_seq, tok_seq, tok_pos, out, out_stride_t, num_tokens,        \
         num_heads, num_kv_heads, dk, dv, rot_dims, window, scale, sinkw, pair_halves, qk_norm_eps, softcap, vcos, vsin,      \
-        out_scale, qnorm_w, prenorm_eps, chunk, vshare, out_f32, (cudaStream_t)stream)))
+        out_scale, qnorm_w, prenorm_eps, chunk, vshare, out_f32, slopes, keep_first, gate_per_head, shared_kv,        \
+        (cudaStream_t)stream)))
     if (dv <= 32) { WA_LAUNCH(1); }
     else if (dv <= 64) { WA_LAUNCH(2); }
     else if (dv <= 128) { WA_LAUNCH(4); }

@@ -73,16 +73,25 @@ class LatentAttentionSpec:
     rot_dim: int
     vdim: int
     kv_rank: int
-    q_rank: int
+    q_rank: int                 # size of the queries' own normed latent; 0: queries are projected directly
     window: int                 # a query at position p sees p - window + 1 .. p; 0 = everything up to p
     rot_base: float
     rot_dims: int               # leading entries of the rotated part that turn (interleaved pairs); the rest pass through
     scale: float
     kv_from: Optional[int]      # layer whose cached latent / rotated key part this layer reads instead of making its own
+    # (factor, original context, fast turns, slow turns), as in WindowAttentionSpec; it acts on the rotated parts only
+    rot_scaling: Optional[tuple] = None
+    sink: bool = False          # the softmax's denominator also contains exp(a learned number per head)
+    gate: str = "head"          # sigmoid gate on the output: "head" (one number per head) or "element"
 
     @property
     def cache_width(self) -> int:
         return self.kv_rank + self.rot_dim
+
+    @property
+    def rot_key(self):
+        """Key of the step's angle tables (TokenInferState.rotary)."""
+        return (self.rot_base, self.rot_dims) if self.rot_scaling is None else (self.rot_base, self.rot_dims, self.rot_scaling)
 
 
 @dataclasses.dataclass(frozen=True)
@@ -117,9 +126,15 @@ class WindowAttentionSpec:
     diff: float = 0.0
     qk_weight_norm: bool = False    # RMS norm with a weight vector of `dim` entries on every query / key part BEFORE rotation
     bias: bool = False              # q, k, v and the output projection have biases
+    distance_bias: bool = False     # score <- score - 2^(-8 (h + 1) / heads) * (query position - key position)
+    keep_first: int = 0             # with a window: the sequence's first positions stay visible
+    gate_per_head: bool = False     # the output gate is one number per head
+    shared_kv: bool = False         # the values are the keys as projected (before their norm); no value projection, no rotation
 
     @property
     def cache_width(self) -> int:
+        if self.shared_kv:          # [1 / rms of every key head, fp32 | keys as projected], both rounded up to 8 entries
+            return (2 * self.kv_heads + 7) // 8 * 8 + (self.kv_heads * self.dim + 7) // 8 * 8
         return self.kv_heads * (self.maps * self.dim + self.vdim)
 
     @property
@@ -142,6 +157,19 @@ class LinearAttentionSpec:
     vdim: int
     decay: tuple
     out_scale: float = 1.0
+
+
+@dataclasses.dataclass(frozen=True)
+class GatedLinearAttentionSpec:
+    """Linear attention with a decay per key channel that depends on the token: alpha = sigmoid(W_a2 (W_a1 h) + b)^(1 / tau);
+    S <- diag(alpha) S + k v^T (dim x vdim per head, fp32, one per sequence), out = S^T (q dim^-1/2), RMS-normed per head (weight of
+    `vdim` entries), gated by silu(W_g h) and projected.  The inner size of W_a2 W_a1 is the checkpoint's.  No cache rows."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    kv_from: Optional[int] = None
+    cache_width: int = 0
 
 
 @dataclasses.dataclass(frozen=True)
@@ -204,6 +232,7 @@ class FeedForwardSpec:
     top: int = 0
     # "relu2": relu(up)^2 | "clamped_glu": min(gate, limit) * sigmoid(1.702 .) * (clamp(up) + 1) | "silu_glu": silu(gate) * up
     # | "gelu_glu": gelu_tanh(gate) * up
+    # ("silu_glu" also as a dense layer)
     activation: str = "relu2"
     limit: float = 0.0          # clamped_glu: bound of the gate (above) and of the up projection (both sides)
     # routing.  "top_softmax": softmax over the `top` largest logits.  "softmax_grouped": scores are a softmax over all experts,
@@ -217,6 +246,7 @@ class FeedForwardSpec:
     shared_ff: int = 0          # hidden size of a shared expert that every token uses (0: none)
     shared_limit: float = 0.0
     shared_gated: bool = False  # the shared expert's output is multiplied by sigmoid(w . h), one number per token
+    bias: bool = False          # the dense layer's three projections have biases
 
 
 def _cache_geometry(mixers):
@@ -529,3 +559,72 @@ class NaforaxModelConfig:
     def load_from_model_path(model_path: str) -> "NaforaxModelConfig":
         with open(os.path.join(model_path, "config.json"), "r", encoding="utf-8") as f:
             return NaforaxModelConfig(json.load(f))
+
+
+# ---------------------------------------------------------------- Zuzezen
+class ZuzezenModelConfig:
+    """config.json of the Zuzezen design: {"architecture": "Zuzezen", "vocab", "width", "norm": {"eps"}, "embedding": {"scale"},
+    "layers": [{"type": "latent_attention" | "attention" | "gla", "mixer": {...}, "mlp": {"kind": "dense", "ff"} | null}, ...]}.
+    "latent_attention": {"heads", "dim", "rot_dim", "vdim", "kv_rank", "scale", "rot": {"base", "dims", "scaling": {"factor",
+    "original", "fast", "slow"}}}; "attention": {"heads", "kv_heads", "dim", "vdim" (= dim), "scale", "mask": {"size",
+    "keep_first"}}; "gla": {"heads", "dim", "vdim", "tau"}.
+    Layers are sequential blocks whose sublayers read the residual stream itself and whose outputs go through an RMS norm (weight
+    stored around zero, applied as 1 + w) and an element-wise scale before they are added.  Every size may differ from layer to
+    layer."""
+    family = "zuzezen"
+
+    def __init__(self, model_config: dict):
+        assert model_config.get("architecture") == "Zuzezen", f"not a Zuzezen config: {model_config.get('architecture')!r}"
+        self.raw = dict(model_config)
+        self.vocab_size = int(model_config["vocab"])
+        self.hidden_size = int(model_config["width"])
+        self.rms_norm_eps = float(model_config["norm"]["eps"])
+        self.embedding_scale = float((model_config.get("embedding") or {}).get("scale", 1.0))
+        self.mixers, self.ffs = [], []
+        for i, layer in enumerate(model_config["layers"]):
+            m = layer["mixer"]
+            if layer["type"] == "latent_attention":
+                rot = m.get("rot") or {}
+                sc = rot.get("scaling")
+                spec = LatentAttentionSpec(
+                    heads=int(m["heads"]), dim=int(m["dim"]), rot_dim=int(m["rot_dim"]), vdim=int(m["vdim"]), kv_rank=int(m["kv_rank"]),
+                    q_rank=0, window=0, rot_base=float(rot.get("base", 10000.0)), rot_dims=int(rot.get("dims", m["rot_dim"])),
+                    scale=float(m["scale"]), kv_from=None,
+                    rot_scaling=(float(sc["factor"]), float(sc["original"]), float(sc["fast"]), float(sc["slow"])) if sc else None,
+                    sink=True, gate="element")
+                assert spec.rot_dims % 2 == 0 and spec.rot_dims <= spec.rot_dim, f"layer {i}: rot.dims must be even and <= rot_dim"
+            elif layer["type"] == "attention":
+                mask = m.get("mask") or {}
+                spec = WindowAttentionSpec(
+                    heads=int(m["heads"]), kv_heads=int(m.get("kv_heads") or m["heads"]), dim=int(m["dim"]), vdim=int(m.get("vdim", m["dim"])),
+                    window=int(mask.get("size", 0)), rot_base=10000.0, rot_dims=0, scale=float(m["scale"]), sink=False, gate=True,
+                    qk_weight_norm=True, bias=True, distance_bias=True, keep_first=int(mask.get("keep_first", 0)), gate_per_head=True,
+                    shared_kv=True)
+                assert spec.heads % spec.kv_heads == 0, f"layer {i}: heads must be a multiple of kv_heads"
+                assert spec.vdim == spec.dim, f"layer {i}: the values are the keys, so vdim must equal dim"
+            else:
+                assert layer["type"] == "gla", f"layer {i}: unknown mixer type {layer['type']!r}"
+                spec = GatedLinearAttentionSpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), tau=float(m["tau"]))
+                assert spec.tau > 0, f"layer {i}: tau must be positive"
+            self.mixers.append(spec)
+            f = layer.get("mlp")
+            if f is None:
+                self.ffs.append(None)
+            else:
+                assert f["kind"] == "dense", f"layer {i}: unknown mlp kind {f['kind']!r}"
+                self.ffs.append(FeedForwardSpec("dense", int(f["ff"]), activation="silu_glu", bias=True))
+        self.num_layers = len(self.mixers)
+        self.cache_slot, self.cache_slots_per_width = _cache_geometry(self.mixers)
+
+    def get_kvslot_size(self, dtype: torch.dtype = torch.bfloat16) -> int:
+        """Bytes of cache one token occupies: one row per attention layer ([latent | rotated key part] or [1 / rms | keys])."""
+        return sum(w * n for w, n in self.cache_slots_per_width.items()) * dtype.itemsize
+
+    def get_state_size(self, dtype: torch.dtype = torch.bfloat16) -> int:
+        """Bytes of recurrent state one SEQUENCE occupies, whatever its length."""
+        return sum(4 * s.heads * s.dim * s.vdim for s in self.mixers if isinstance(s, GatedLinearAttentionSpec))
+
+    @staticmethod
+    def load_from_model_path(model_path: str) -> "ZuzezenModelConfig":
+        with open(os.path.join(model_path, "config.json"), "r", encoding="utf-8") as f:
+            return ZuzezenModelConfig(json.load(f))

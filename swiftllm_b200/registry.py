@@ -6,6 +6,7 @@
     rivudra     "architecture": "Rivudra"                   RivudraModelConfig     worker.rivudra_model.RivudraModel
     buzarax     "architecture": "Buzarax"                   BuzaraxModelConfig     worker.buzarax_model.BuzaraxModel
     naforax     "architecture": "Naforax"                   NaforaxModelConfig     worker.naforax_model.NaforaxModel
+    zuzezen     "architecture": "Zuzezen"                   ZuzezenModelConfig     worker.zuzezen_model.ZuzezenModel
 
 Every worker class has the same public surface (load_weights, profile_num_blocks, init_kvcache_and_swap, forward /
 forward_async with the prefill-chunks-then-decodes batch layout, free_seqs_resources), so schedulers, examples and
@@ -29,6 +30,8 @@ _FAMILIES = {
                 "swiftllm_b200.model_config:BuzaraxModelConfig", "swiftllm_b200.worker.buzarax_model:BuzaraxModel"),
     "naforax": (lambda raw: raw.get("architecture") == "Naforax",
                 "swiftllm_b200.model_config:NaforaxModelConfig", "swiftllm_b200.worker.naforax_model:NaforaxModel"),
+    "zuzezen": (lambda raw: raw.get("architecture") == "Zuzezen",
+                "swiftllm_b200.model_config:ZuzezenModelConfig", "swiftllm_b200.worker.zuzezen_model:ZuzezenModel"),
 }
 
 

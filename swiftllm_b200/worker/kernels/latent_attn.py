@@ -36,14 +36,17 @@ def _num_splits(T: int, H: int, window: int, dtype) -> int:
 
 
 def latent_attention(q_lat: torch.Tensor, q_rot: torch.Tensor, gate, cache: torch.Tensor, slot: int, block_table: torch.Tensor,
-                     infer_state, out: torch.Tensor, rot_dims: int, window: int, scale: float, cos: torch.Tensor, sin: torch.Tensor):
+                     infer_state, out: torch.Tensor, rot_dims: int, window: int, scale: float, cos: torch.Tensor, sin: torch.Tensor,
+                     sink: torch.Tensor = None):
     """q_lat [T, H, r], q_rot [T, H, dr] (un-rotated), gate [T, H] logits or None, out [T, H, r]; views with arbitrary token /
-    head strides are taken as they are (the innermost stride must be 1)."""
+    head strides are taken as they are (the innermost stride must be 1).  sink fp32 [H] or None: exp(sink[h]) joins the softmax's
+    denominator."""
     T, H, r = q_lat.shape
     dr = q_rot.shape[2]
     assert q_lat.stride(2) == 1 and q_rot.stride(2) == 1 and out.stride(2) == 1 and out.shape == q_lat.shape
     assert cache.shape[3] == r + dr and cache.dtype == q_lat.dtype
     assert gate is None or (gate.shape == (T, H) and gate.stride(1) == 1)
+    assert sink is None or (sink.dtype == torch.float32 and sink.shape == (H,) and sink.is_contiguous())
     _lib.require_device(q_lat)
     nsplit = _num_splits(T, H, window, q_lat.dtype)
     ws = torch.empty((T, H, nsplit, r + 2), dtype=torch.float32, device=q_lat.device) if nsplit > 1 else None
@@ -52,5 +55,5 @@ def latent_attention(q_lat: torch.Tensor, q_rot: torch.Tensor, gate, cache: torc
         _lib.ptr(cos), _lib.ptr(sin), _lib.ptr(gate), gate.stride(0) if gate is not None else 0,
         cache.data_ptr(), cache.shape[1], slot, cache.shape[2], block_table.data_ptr(), block_table.shape[1],
         infer_state.token_seq_ids.data_ptr(), infer_state.token_positions.data_ptr(),
-        out.data_ptr(), out.stride(0), out.stride(1), T, H, r, dr, rot_dims, window, scale, nsplit, _lib.ptr(ws),
+        out.data_ptr(), out.stride(0), out.stride(1), T, H, r, dr, rot_dims, window, scale, _lib.ptr(sink), nsplit, _lib.ptr(ws),
         _lib.dtype_tag_f32(q_lat.dtype), _lib.stream()), "latent_attention")

@@ -10,6 +10,11 @@ def linear(
     return torch.nn.functional.linear(a, w)
 
 
+def linear_bias(a: torch.Tensor, w: torch.Tensor, b) -> torch.Tensor:
+    """a w^T + b (b [c] or None)."""
+    return torch.nn.functional.linear(a, w, b)
+
+
 def linear_f32_out(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     """a [n, k] (row-strided allowed), w [m, k] in a's dtype -> a w^T as fp32 [n, m]: the library GEMM's fp32 accumulator is
     written out unrounded (inputs that feed a recurrence's step size or decay)."""

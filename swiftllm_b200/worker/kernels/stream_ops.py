@@ -1,6 +1,6 @@
 """Kernels of sequential decoder blocks on an fp32 residual stream whose sublayer outputs are normalised before they are added
 (csrc/stream_ops.cu): the embedding with a hashed table of token pairs, the post-norm add with the weighted sum over depth, the
-tanh cap, and the sigmoid router with the SiLU-gated expert activation.  The stream, norms and the router are fp32 for every
+tanh cap, the sigmoid router with the SiLU-gated expert activation, the SiLU gated linear unit and the element-wise sigmoid gate.  The stream, norms and the router are fp32 for every
 storage dtype of the projections."""
 import torch
 
@@ -8,8 +8,8 @@ from swiftllm_b200 import _lib
 
 
 def embed_pair_hash(tokens: torch.Tensor, infer_state, last_token: torch.Tensor, embed: torch.Tensor, pairs, buckets: int,
-                    mul_prev: int, mul_cur: int, x_copy: torch.Tensor = None):
-    """-> (x fp32 [T, W], h [T, W] in embed's dtype).  x = embed[token] + pairs[hash(previous token, token)] (pairs may be None);
+                    mul_prev: int, mul_cur: int, x_copy: torch.Tensor = None, scale: float = 1.0):
+    """-> (x fp32 [T, W], h [T, W] in embed's dtype).  x = embed[token] * scale + pairs[hash(previous token, token)] (pairs may be None);
     the previous token of a step's first row comes from last_token[sequence row], which is then moved on to the step's last
     token.  x_copy (fp32 [T, W]) receives the same values."""
     _lib.require_device(embed)
@@ -20,7 +20,7 @@ def embed_pair_hash(tokens: torch.Tensor, infer_state, last_token: torch.Tensor,
     st = infer_state
     _lib.check(_lib.lib().sllm_embed_pair_hash(
         tokens.data_ptr(), st.token_seq_ids.data_ptr(), st.token_positions.data_ptr(), _lib.ptr(last_token), embed.data_ptr(),
-        _lib.ptr(pairs), buckets, mul_prev, mul_cur, x.data_ptr(), _lib.ptr(x_copy), h.data_ptr(), T, W,
+        _lib.ptr(pairs), buckets, mul_prev, mul_cur, scale, x.data_ptr(), _lib.ptr(x_copy), h.data_ptr(), T, W,
         _lib.dtype_tag_f32(embed.dtype), _lib.stream()), "embed_pair_hash")
     if pairs is not None:
         _lib.check(_lib.lib().sllm_store_last_tokens(tokens.data_ptr(), st.seg_starts.data_ptr(), st.seq_ids.data_ptr(),
@@ -30,16 +30,37 @@ def embed_pair_hash(tokens: torch.Tensor, infer_state, last_token: torch.Tensor,
 
 def postnorm_add_mix(x: torch.Tensor, y, gain, eps: float, h: torch.Tensor, history: torch.Tensor = None, slot: int = 0,
                      mix: torch.Tensor = None):
-    """x (fp32 [T, W], in place) <- x + gain * y / rms(y)  (y None: unchanged); with `history` (fp32 [slots, T, W]) the result is
+    """x (fp32 [T, W], in place) <- x + gain * y / rms(y)  (y None: unchanged; gain fp32 [1] or [W]); with `history` (fp32 [slots, T, W]) the result is
     kept in history[slot], and with `mix` (fp32 [slot + 1]) x <- sum_j mix[j] * history[j].  h <- x rounded to h's dtype."""
     assert x.dtype == torch.float32 and x.is_contiguous() and h.is_contiguous() and h.shape == x.shape
     assert y is None or (y.dtype == h.dtype and y.is_contiguous() and y.shape == x.shape and gain.dtype == torch.float32)
     assert history is None or (history.dtype == torch.float32 and history.is_contiguous() and history.shape[1:] == x.shape)
     assert mix is None or (history is not None and mix.dtype == torch.float32 and mix.numel() == slot + 1 and slot < history.shape[0])
     _lib.require_device(x)
-    _lib.check(_lib.lib().sllm_postnorm_add_mix(x.data_ptr(), _lib.ptr(y), _lib.ptr(gain), eps, _lib.ptr(history), slot, _lib.ptr(mix),
+    assert gain is None or gain.numel() in (1, x.shape[1])
+    per_channel = 1 if gain is not None and gain.numel() > 1 else 0
+    _lib.check(_lib.lib().sllm_postnorm_add_mix(x.data_ptr(), _lib.ptr(y), _lib.ptr(gain), per_channel, eps, _lib.ptr(history), slot, _lib.ptr(mix),
                                                 h.data_ptr(), x.shape[0], x.shape[1], _lib.dtype_tag_f32(h.dtype), _lib.stream()),
                "postnorm_add_mix")
+
+
+def silu_glu(u: torch.Tensor) -> torch.Tensor:
+    """u [T, 2 F] = [gate | up] -> silu(gate) * up [T, F]."""
+    assert u.is_contiguous() and u.shape[1] % 2 == 0
+    _lib.require_device(u)
+    T, F = u.shape[0], u.shape[1] // 2
+    y = torch.empty((T, F), dtype=u.dtype, device=u.device)
+    _lib.check(_lib.lib().sllm_silu_glu(u.data_ptr(), y.data_ptr(), T, F, _lib.dtype_tag_f32(u.dtype), _lib.stream()), "silu_glu")
+    return y
+
+
+def sigmoid_gate_inplace(x: torch.Tensor, gate: torch.Tensor):
+    """x [T, n] *= sigmoid(gate) (gate: logits [T, n], a row-strided slice is fine)."""
+    T, n = x.shape
+    assert x.is_contiguous() and gate.shape == x.shape and gate.stride(1) == 1 and gate.dtype == x.dtype
+    _lib.require_device(x)
+    _lib.check(_lib.lib().sllm_sigmoid_gate_inplace(x.data_ptr(), gate.data_ptr(), gate.stride(0) if T > 1 else max(gate.stride(0), n),
+                                                    T, n, _lib.dtype_tag_f32(x.dtype), _lib.stream()), "sigmoid_gate_inplace")
 
 
 def tanh_cap_inplace(x: torch.Tensor, cap: float):

@@ -4,7 +4,8 @@
 Options (`AttnOptions`) that other designs switch on: rotary pairs as halves instead of neighbours, unit-RMS queries and keys, a
 tanh cap on the scores, values that are stored turned by their position (the output is turned back), a factor on the output, an
 RMS norm with weight on every query / key head before it turns, a chunked mask, several key heads (score maps) per value head
-with fp32 output, and `diff_combine`, which turns two maps' outputs into one gated head."""
+with fp32 output, and `diff_combine`, which turns two maps' outputs into one gated head; a bias on the distance, kept first
+positions beside the window, one gate per head, and values that are the un-normed keys (`shared_kv_store`)."""
 import dataclasses
 import torch
 
@@ -23,9 +24,20 @@ class AttnOptions:
     chunk: int = 0                  # > 0: a query at position p sees only positions >= floor(p / chunk) * chunk
     vshare: int = 1                 # this many neighbouring key heads share one value head (cache row: G keys, G / vshare values)
     out_f32: bool = False           # the attention output is fp32 whatever the storage dtype
+    slopes: object = None           # fp32 [H]: score <- score - slopes[h] * (query position - key position)
+    keep_first: int = 0             # > 0: with a window, the sequence's first positions stay visible
+    gate_per_head: bool = False     # gate logits [T, H] instead of [T, H * dv]
+    # the values are the un-normed keys: a cache row is [1 / rms of every key head (fp32) | keys as projected], `shared_row_width`
+    # entries wide; the weight of the keys' norm is part of q_norm
+    shared_kv: bool = False
 
 
 PLAIN = AttnOptions()
+
+
+def shared_row_width(kv_heads: int, dk: int) -> int:
+    """Entries of a cache row whose keys are also the values: 2 per key head for the fp32 norm, then the keys, both rounded up to 8."""
+    return (2 * kv_heads + 7) // 8 * 8 + (kv_heads * dk + 7) // 8 * 8
 
 
 def _stride0(x: torch.Tensor) -> int:
@@ -51,6 +63,19 @@ def window_kv_store(k: torch.Tensor, v: torch.Tensor, cache: torch.Tensor, slot:
         "window_kv_store")
 
 
+def shared_kv_store(k: torch.Tensor, cache: torch.Tensor, slot: int, block_table: torch.Tensor, infer_state, kv_heads: int, dk: int,
+                    eps: float):
+    """k [T, G * dk] as projected (a row-strided slice is fine) -> the tokens' cache rows [1 / rms | k] (AttnOptions.shared_kv)."""
+    T = k.shape[0]
+    assert k.dim() == 2 and k.stride(1) == 1 and k.shape[1] == kv_heads * dk
+    assert cache.is_contiguous() and cache.dtype == k.dtype and cache.shape[3] == shared_row_width(kv_heads, dk)
+    _lib.require_device(k)
+    _lib.check(_lib.lib().sllm_shared_kv_store(
+        k.data_ptr(), _stride0(k), infer_state.token_seq_ids.data_ptr(), infer_state.token_positions.data_ptr(), block_table.data_ptr(),
+        block_table.shape[1], cache.data_ptr(), cache.shape[1], slot, cache.shape[2], T, kv_heads, dk, eps,
+        _lib.dtype_tag_f32(k.dtype), _lib.stream()), "shared_kv_store")
+
+
 def window_attention(q: torch.Tensor, gate, cache: torch.Tensor, slot: int, block_table: torch.Tensor, infer_state,
                      out: torch.Tensor, heads: int, kv_heads: int, dk: int, dv: int, rot_dims: int, window: int, scale: float,
                      sink: bool, cos: torch.Tensor, sin: torch.Tensor, opt: AttnOptions = PLAIN, vcos: torch.Tensor = None,
@@ -59,8 +84,10 @@ def window_attention(q: torch.Tensor, gate, cache: torch.Tensor, slot: int, bloc
     are fine."""
     T = q.shape[0]
     assert q.stride(1) == 1 and out.stride(1) == 1 and q.shape == (T, heads * dk) and out.shape == (T, heads * dv)
-    assert gate is None or (gate.shape == (T, heads * dv) and gate.stride(1) == 1 and gate.dtype == q.dtype)
-    assert cache.shape[3] == kv_heads * dk + kv_heads // opt.vshare * dv and cache.dtype == q.dtype
+    assert gate is None or (gate.shape == (T, heads if opt.gate_per_head else heads * dv) and gate.stride(1) == 1 and gate.dtype == q.dtype)
+    row = shared_row_width(kv_heads, dk) if opt.shared_kv else kv_heads * dk + kv_heads // opt.vshare * dv
+    assert cache.shape[3] == row and cache.dtype == q.dtype and (not opt.shared_kv or dk == dv)
+    assert opt.slopes is None or (opt.slopes.dtype == torch.float32 and opt.slopes.shape == (heads,))
     assert out.dtype == (torch.float32 if opt.out_f32 else q.dtype)
     assert opt.q_norm is None or (opt.q_norm.dtype == torch.float32 and opt.q_norm.shape == (dk,))
     _lib.require_device(q)
@@ -70,7 +97,8 @@ def window_attention(q: torch.Tensor, gate, cache: torch.Tensor, slot: int, bloc
         infer_state.token_seq_ids.data_ptr(), infer_state.token_positions.data_ptr(), out.data_ptr(), _stride0(out), T,
         min(T, max(0, int(getattr(infer_state, "num_prefill_tokens", T)))), heads, kv_heads, dk, dv, rot_dims, window, scale, 1 if sink else 0,
         1 if opt.pair_halves else 0, opt.qk_norm_eps, opt.softcap, _lib.ptr(vcos), _lib.ptr(vsin), opt.out_scale,
-        _lib.ptr(opt.q_norm), opt.prenorm_eps, opt.chunk, opt.vshare, 1 if opt.out_f32 else 0, _lib.dtype_tag_f32(q.dtype),
+        _lib.ptr(opt.q_norm), opt.prenorm_eps, opt.chunk, opt.vshare, 1 if opt.out_f32 else 0,
+        _lib.ptr(opt.slopes), opt.keep_first, 1 if opt.gate_per_head else 0, 1 if opt.shared_kv else 0, _lib.dtype_tag_f32(q.dtype),
         _lib.stream()),
         "window_attention")
 

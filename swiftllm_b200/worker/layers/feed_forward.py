@@ -1,5 +1,5 @@
 """Feed-forward sublayers: dense and mixture-of-experts with the squared-ReLU activation, a dense clamped gated linear unit, a
-dense GELU gated linear unit, a mixture of clamped gated-linear-unit experts (group-limited routing with renormalised scores, or
+dense GELU gated linear unit, a dense SiLU gated linear unit with biases, a mixture of clamped gated-linear-unit experts (group-limited routing with renormalised scores, or
 the plain softmax scores of the largest experts) with a shared expert that may have a per-token sigmoid weight, and a mixture of
 SiLU-gated experts routed by sigmoid scores with a bias that only takes part in the choice.
 
@@ -15,11 +15,11 @@ only matters once the step is compute-bound (a decode step streams every expert'
 tokens * top >= experts)."""
 import torch
 
-from swiftllm_b200.worker.kernels.linear import linear
+from swiftllm_b200.worker.kernels.linear import linear, linear_bias
 from swiftllm_b200.worker.kernels.parallel_block import (moe_clamped_glu_scale, moe_relu2_scale_inplace, moe_route,
                                                          moe_route_grouped, relu2_inplace)
 from swiftllm_b200.worker.kernels.sandwich_ops import gelu_glu, moe_route_softmax
-from swiftllm_b200.worker.kernels.stream_ops import moe_route_sigmoid, moe_silu_glu_scale
+from swiftllm_b200.worker.kernels.stream_ops import moe_route_sigmoid, moe_silu_glu_scale, silu_glu
 
 GLU_SIGMOID_SLOPE = 1.702       # the gate's activation is g * sigmoid(1.702 g)
 ROUTE_NORM_EPS = 1e-20          # added to the sum of the chosen scores before dividing by it
@@ -95,6 +95,19 @@ class GeluGluFeedForward:
         return linear(gelu_glu(linear(h, self.weight.up)), self.weight.down)
 
 
+class SiluGluFeedForward:
+    """Dense silu(gate) * up -> down, with biases where the specification has them: ONE [gate | up] GEMM, the activation kernel, ONE
+    down GEMM."""
+
+    def __init__(self, spec, weight):
+        self.spec, self.weight = spec, weight
+
+    def forward(self, h: torch.Tensor, x32=None) -> torch.Tensor:
+        w = self.weight
+        up_b, down_b = (w.up_bias, w.down_bias) if self.spec.bias else (None, None)
+        return linear_bias(silu_glu(linear_bias(h, w.up, up_b)), w.down, down_b)
+
+
 class SiluGluMixtureOfExperts:
     """Experts y = silu(gate) * up -> down, no biases.  Routing: scores are sigmoids of fp32 router logits; the `top` experts with
     the largest score + correction are chosen and weighted by their plain scores (not renormalised).  Dense formulation as above:
@@ -116,6 +129,9 @@ class SiluGluMixtureOfExperts:
 def build_feed_forward(spec, weight):
     if spec is None:
         return None
+    if spec.activation == "silu_glu" and spec.kind == "dense":
+        return SiluGluFeedForward(spec, weight)
+    assert not spec.bias, "only the dense SiLU gated linear unit has biases"
     if spec.activation == "silu_glu":
         assert spec.kind == "moe" and spec.routing == "sigmoid_bias"
         return SiluGluMixtureOfExperts(spec, weight)

@@ -16,6 +16,6 @@ class ParallelBlockLayer:
         self.ff = build_feed_forward(model_config.ffs[layer_id], weight)
 
     def forward(self, h, caches, block_table, infer_state):
-        y_mix = self.mixer.forward(h, caches, block_table, infer_state)
+        y_mix = self.mixer.forward(h, caches, block_table, None, infer_state)
         y_ff = self.ff.forward(h) if self.ff is not None else None
         return y_mix, y_ff

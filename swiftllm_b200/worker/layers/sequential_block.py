@@ -1,12 +1,16 @@
 """A sequential decoder block whose sublayers read the residual stream itself and whose OUTPUTS are normalised before they are
-added: x <- x + g1 * rms(mixer(x)), then x <- x + g2 * rms(ff(x)) (scalar gains).  The block returns nothing: it updates the
+added: x <- x + g1 * rms(mixer(x)), then x <- x + g2 * rms(ff(x)) (scalar gains, or one per channel).  The block returns nothing: it updates the
 fp32 stream `x` and its rounding `h` (what the projections read) in place; the second update also applies the weighted sum over
 the results of all earlier layers when the design has one (worker/kernels/stream_ops.py)."""
-from swiftllm_b200.model_config import GatedRecurrenceSpec, ParallelMixerSpec
+from swiftllm_b200.model_config import (GatedLinearAttentionSpec, GatedRecurrenceSpec, LatentAttentionSpec, ParallelMixerSpec,
+                                        WindowAttentionSpec)
 from swiftllm_b200.worker.kernels.stream_ops import postnorm_add_mix
 from swiftllm_b200.worker.layers.feed_forward import build_feed_forward
+from swiftllm_b200.worker.layers.gated_linear_attention import GatedLinearAttentionMixer
 from swiftllm_b200.worker.layers.gated_recurrence import GatedRecurrenceMixer
+from swiftllm_b200.worker.layers.latent_attention import LatentAttentionMixer
 from swiftllm_b200.worker.layers.parallel_mixer import ParallelMixer
+from swiftllm_b200.worker.layers.window_attention import SharedKeyValueAttentionMixer
 
 
 class PostNormBlockLayer:
@@ -15,6 +19,12 @@ class PostNormBlockLayer:
         spec = model_config.mixers[layer_id]
         if isinstance(spec, GatedRecurrenceSpec):
             self.mixer = GatedRecurrenceMixer(spec, weight, layer_id)
+        elif isinstance(spec, GatedLinearAttentionSpec):
+            self.mixer = GatedLinearAttentionMixer(spec, weight, self.eps, layer_id)
+        elif isinstance(spec, LatentAttentionSpec):
+            self.mixer = LatentAttentionMixer(spec, weight, self.eps, model_config.cache_slot[layer_id])
+        elif isinstance(spec, WindowAttentionSpec):
+            self.mixer = SharedKeyValueAttentionMixer(spec, weight, self.eps, model_config.cache_slot[layer_id])
         else:
             assert isinstance(spec, ParallelMixerSpec)
             self.mixer = ParallelMixer(spec, weight, self.eps, model_config.cache_slot[layer_id], layer_id)

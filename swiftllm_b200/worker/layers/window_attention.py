@@ -4,13 +4,18 @@ sigmoid output gate: one kernel) -> o GEMM.  The specification's options (model_
 halves, stretched frequencies, unit-RMS queries and keys, capped scores, values turned by their position) go to the same two
 kernels.  `attend` is the part between the two GEMMs, for mixers that fuse their projections with a neighbour's.
 
+`SharedKeyValueAttentionMixer`: the values are the keys as projected, so there is ONE fused GEMM with bias [q ; k ; gate per head],
+the cache holds the un-normed keys with their 1 / rms, and one staged tile serves the attention kernel as keys and values; scores
+carry a bias on the distance; the first positions of the sequence stay visible beside the window.
+
 `DifferentialAttentionMixer`: two score maps per head over the same values.  Every map is a query head of its own for the same two
 kernels (twice the heads, `vshare` = 2 key heads per value head, fp32 output); one more kernel subtracts the maps, normalises
 the head and applies the gate."""
 import torch
 
-from swiftllm_b200.worker.kernels.linear import linear
-from swiftllm_b200.worker.kernels.window_attn import AttnOptions, diff_combine, window_attention, window_kv_store
+from swiftllm_b200.worker.kernels.linear import linear, linear_bias
+from swiftllm_b200.worker.kernels.window_attn import (AttnOptions, diff_combine, shared_kv_store, window_attention,
+                                                      window_kv_store)
 
 
 class WindowAttentionMixer:
@@ -46,12 +51,51 @@ class WindowAttentionMixer:
         window_attention(q, gate, cache, self.cache_slot, block_table, st, out, m.heads, m.kv_heads, m.dim, m.vdim,
                          m.rot_dims, m.window, m.scale, m.sink, cos, sin, self.options, vcos, vsin)
 
-    def forward(self, h: torch.Tensor, caches: dict, block_table: torch.Tensor, st) -> torch.Tensor:
+    def forward(self, h: torch.Tensor, caches: dict, block_table: torch.Tensor, states, st) -> torch.Tensor:
         m, w = self.spec, self.weight
         proj = linear(h, w.in_proj)                             # [T, H dk | G dk | G dv (| H dv)]
         parts = list(torch.split(proj, self.proj_widths, dim=1)) + [None]
         out = torch.empty((h.shape[0], m.heads * m.vdim), dtype=h.dtype, device=h.device)
         self.attend(parts[0], parts[1], parts[2], parts[3], out, caches, block_table, st)
+        return linear(out, w.o)
+
+
+def distance_slopes(heads: int) -> list:
+    """Slope of every head's bias on the distance: 2^(-8 (h + 1) / heads)."""
+    return [2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)]
+
+
+class SharedKeyValueAttentionMixer:
+    """ONE GEMM with bias [q ; k ; gate] -> 1 / rms of the keys + cache store (one kernel) -> attention (RMS norm of q with the
+    product of both norms' weights, window + kept first positions, bias on the distance, softmax, gate per head: one kernel) ->
+    o GEMM.  (q^ . (k / rms(k) * w_k) = (q^ * w_k) . k / rms(k): the cached row needs no weight.)"""
+
+    def __init__(self, spec, weight, eps: float, cache_key):
+        assert spec.shared_kv and spec.qk_weight_norm and spec.gate_per_head and spec.rot_dims == 0 and not spec.sink
+        self.spec, self.weight, self.eps = spec, weight, eps
+        self.cache_width, self.cache_slot = cache_key
+        slopes = None
+        if spec.distance_bias:
+            slopes = torch.tensor(distance_slopes(spec.heads), dtype=torch.float32).to(weight.qk_norm.device)
+        self.options = AttnOptions(q_norm=weight.qk_norm, prenorm_eps=eps, slopes=slopes, keep_first=spec.keep_first,
+                                   gate_per_head=True, shared_kv=True)
+
+    def register(self, model):
+        pass
+
+    def state_layout(self) -> dict:
+        return {}
+
+    def forward(self, h: torch.Tensor, caches: dict, block_table: torch.Tensor, states, st) -> torch.Tensor:
+        m, w = self.spec, self.weight
+        q, k, gate = torch.split(linear_bias(h, w.in_proj, w.in_bias), [m.heads * m.dim, m.kv_heads * m.dim, m.heads], dim=1)
+        out = torch.empty((h.shape[0], m.heads * m.dim), dtype=h.dtype, device=h.device)
+        if st.ignore_kvcache:
+            return linear(out.zero_(), w.o)
+        cache = caches[self.cache_width]
+        shared_kv_store(k, cache, self.cache_slot, block_table, st, m.kv_heads, m.dim, self.eps)
+        window_attention(q, gate, cache, self.cache_slot, block_table, st, out, m.heads, m.kv_heads, m.dim, m.dim, 0, m.window, m.scale,
+                         False, None, None, self.options)
         return linear(out, w.o)
 
 

@@ -410,6 +410,95 @@ def load_naforax_weights(model_config, dtype: torch.dtype, model_path: Optional[
     return weight
 
 
+class ZuzezenLayerWeight:
+    """One sequential block.  Checkpoint names: `l<i>.{norm1, ls1}` (and `norm2, ls2` with a feed-forward), and
+    mixer "latent_attention": `l<i>.mix.{q, dkv, dkv.norm, uk, uv, sink, g, o}`;
+    mixer "attention": `l<i>.mix.{q, q.b, k, k.b, q.norm, k.norm, g, o}`;
+    mixer "gla": `l<i>.mix.{q, k, v, g, a1, a2, a2.b, norm, o}`;
+    feed-forward: `l<i>.mlp.{gate, gate.b, up, up.b, down, down.b}`.
+    Fusions made at load time: every projection that reads the block's input is one GEMM operand (`in_proj`: [q ; g ; dkv],
+    [q ; k ; g] with `in_bias`, [q ; k ; v ; g ; a1]); the output norm's 1 + w and the layer scale are one fp32 gain per channel
+    (`norm1`, `norm2`); both norms of the attention mixer are one fp32 weight on the query (`qk_norm`); [gate ; up] is one operand.
+    The inner size of the decay projection (a1 rows, a2 columns) is the checkpoint's; weight sources that make tensors up (getters
+    that honour the requested shape) get DECAY_RANK."""
+
+    DECAY_RANK = 16
+
+    def __init__(self, layer_id: int, model_config, dtype: torch.dtype):
+        self.layer_id, self.model_config, self.dtype = layer_id, model_config, dtype
+
+    def load_weights(self, getter: Callable, device):
+        from swiftllm_b200.model_config import GatedLinearAttentionSpec, LatentAttentionSpec
+        c, i, f32 = self.model_config, self.layer_id, torch.float32
+        m, f, W = c.mixers[i], c.ffs[i], c.hidden_size
+
+        def get(name, shape, dtype=None):
+            w = getter(f"l{i}.{name}", tuple(self.DECAY_RANK if s is None else s for s in shape), dtype or self.dtype)
+            assert isinstance(w, torch.Tensor) and w.dim() == len(shape) and all(s in (None, n) for s, n in zip(shape, w.shape)), \
+                f"l{i}.{name}: expected shape {tuple(shape)}"
+            return w.to(device=device, dtype=dtype or self.dtype).contiguous()
+
+        def gain(norm, scale):
+            return (unit_offset_norm(get(norm, (W,), f32)) * get(scale, (W,), f32)).contiguous()
+
+        self.norm1 = gain("norm1", "ls1")
+        if isinstance(m, LatentAttentionSpec):
+            H, r = m.heads, m.kv_rank
+            self.in_proj = torch.cat([get("mix.q", (H * (m.dim + m.rot_dim), W)), get("mix.g", (H * m.vdim, W)),
+                                      get("mix.dkv", (m.cache_width, W))], dim=0).contiguous()
+            self.dkv_norm = get("mix.dkv.norm", (r,))
+            self.uk = get("mix.uk", (H * m.dim, r)).view(H, m.dim, r)
+            self.uv = get("mix.uv", (H * m.vdim, r)).view(H, m.vdim, r)
+            self.sink = get("mix.sink", (H,), f32)
+            self.o = get("mix.o", (W, H * m.vdim))
+        elif isinstance(m, GatedLinearAttentionSpec):
+            nk, nv = m.heads * m.dim, m.heads * m.vdim
+            a1 = get("mix.a1", (None, W))
+            self.in_proj = torch.cat([get("mix.q", (nk, W)), get("mix.k", (nk, W)), get("mix.v", (nv, W)), get("mix.g", (nv, W)), a1],
+                                     dim=0).contiguous()
+            self.a2, self.a2_bias = get("mix.a2", (nk, a1.shape[0])), get("mix.a2.b", (nk,), f32)
+            self.head_norm = get("mix.norm", (m.vdim,), f32)
+            self.o = get("mix.o", (W, nv))
+        else:
+            H, G, d = m.heads, m.kv_heads, m.dim
+            self.in_proj = torch.cat([get("mix.q", (H * d, W)), get("mix.k", (G * d, W)), get("mix.g", (H, W))], dim=0).contiguous()
+            self.in_bias = torch.cat([get("mix.q.b", (H * d,)), get("mix.k.b", (G * d,)),
+                                      torch.zeros((H,), dtype=self.dtype, device=device)]).contiguous()
+            self.qk_norm = (get("mix.q.norm", (d,), f32) * get("mix.k.norm", (d,), f32)).contiguous()
+            self.o = get("mix.o", (W, H * d))
+        if f is None:
+            return
+        self.norm2 = gain("norm2", "ls2")
+        self.up = torch.cat([get("mlp.gate", (f.ff, W)), get("mlp.up", (f.ff, W))], dim=0).contiguous()
+        self.up_bias = torch.cat([get("mlp.gate.b", (f.ff,)), get("mlp.up.b", (f.ff,))]).contiguous()
+        self.down, self.down_bias = get("mlp.down", (W, f.ff)), get("mlp.down.b", (W,))
+
+
+class ZuzezenWeight:
+    def __init__(self, model_config, dtype: torch.dtype):
+        self.model_config, self.dtype = model_config, dtype
+        self.layers = [ZuzezenLayerWeight(i, model_config, dtype) for i in range(model_config.num_layers)]
+
+    def load_weights(self, getter: Callable, device="cuda"):
+        c = self.model_config
+        vs = (c.vocab_size, c.hidden_size)
+        self.wte = getter("embed", vs, self.dtype).to(device=device, dtype=self.dtype).contiguous()
+        self.final_norm = unit_offset_norm(getter("final.norm", (c.hidden_size,), torch.float32).to(device=device))
+        self.lm_head = getter("head", vs, self.dtype).to(device=device, dtype=self.dtype).contiguous()
+        self.lm_head_sharded = False
+        for layer in self.layers:
+            layer.load_weights(getter, device)
+
+
+def load_zuzezen_weights(model_config, dtype: torch.dtype, model_path: Optional[str], use_dummy: bool = False,
+                         getter: Optional[Callable] = None, device="cuda") -> ZuzezenWeight:
+    if getter is None:
+        getter = dummy_getter(device) if use_dummy else checkpoint_getter(model_path, device)
+    weight = ZuzezenWeight(model_config, dtype)
+    weight.load_weights(getter, device)
+    return weight
+
+
 # ---------------------------------------------------------------- getters
 def dummy_getter(device="cuda"):
     """weight.py:215-218: uniform(-1e-3, 1e-3), unseeded ("mainly for profiling")."""
