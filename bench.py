@@ -4,7 +4,7 @@
   python bench.py [--gpus N] [--steps K] [--warmup W]            # this implementation
   python bench.py --impl reference ...                            # CPU arm: torch-eager oracle port on host cores
   torchrun --nproc-per-node N bench.py --gpus N ...               # N > 1: tensor parallel (heads / FFN columns)
-  python bench.py --arch-compare all [--steps K] [--warmup W]     # NOT the headline: Bupozen / Rivudra / Buzarax / Naforax workers beside the Llama worker
+  python bench.py --arch-compare all [--steps K] [--warmup W]     # NOT the headline: Bupozen / Rivudra / Buzarax / Naforax / Zuzezen workers beside the Llama worker
                                                                   # (prefill / decode tok/s, attention roofline), 1 GPU
 
 Workload: Llama-3-8B shapes, bf16, pure decode, batch 256, every sequence at
@@ -88,7 +88,7 @@ def parse():
     ap.add_argument("--no-live-traffic", action="store_true", help="skip the ncu DRAM-byte measurement of the decode kernel")
     ap.add_argument("--no-prefill", action="store_true")
     ap.add_argument("--arch-models", type=str, default="", metavar="NAMES",
-                    help="with --arch-compare: only these workers (comma-separated: bupozen, rivudra, buzarax, naforax, llama); default all")
+                    help="with --arch-compare: only these workers (comma-separated: bupozen, rivudra, buzarax, naforax, zuzezen, llama); default all")
     ap.add_argument("--arch-compare", type=str, default="", metavar="SIZES",
                     help="instead of the headline workload: prefill and decode throughput of the Bupozen and Rivudra workers beside the "
                          "Llama worker at equal width / depth (random weights), with the attention kernels' roofline fractions; "
@@ -166,14 +166,25 @@ def _arch_models(sz, dtype, only=None):
            "logit_softcap": 30.0, "canon": {"taps": 4}, "loop": {"start": 1, "stop": 3, "times": 1},
            "layers": [{"type": naf_mixers[i % 4][0], "mixer": naf_mixers[i % 4][1],
                        "mlp": {"kind": "dense", "ff": sz["ff"]} if i == 0 else naf_moe} for i in range(sz["layers"])]}
-    for name, raw in (("bupozen", bup), ("rivudra", riv), ("buzarax", buz), ("naforax", naf), ("llama", llama)):
+    # Zuzezen: [latent attention (128 + 64 per head, 512-wide latent, full causal) + dense ff], [windowed attention (heads / 4 key
+    # heads of W / H entries that are also the values, 4 kept positions) + dense ff], [gated linear attention (128 x 128 state per head),
+    # no ff], [latent attention + dense ff]
+    zlat = {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5,
+            "rot": {"base": 50000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 4096, "fast": 24.0, "slow": 2.0}}}
+    zwin = {"heads": H, "kv_heads": G, "dim": W // H, "vdim": W // H, "scale": (W // H) ** -0.5, "mask": {"size": sz["window"], "keep_first": 4}}
+    zuz_mixers = [("latent_attention", zlat), ("attention", zwin), ("gla", {"heads": H, "dim": 128, "vdim": 128, "tau": 16.0}),
+                  ("latent_attention", zlat)]
+    zuz = {"architecture": "Zuzezen", "vocab": sz["vocab"], "width": W, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+           "layers": [{"type": zuz_mixers[i % 4][0], "mixer": zuz_mixers[i % 4][1],
+                       "mlp": None if i % 4 == 2 else {"kind": "dense", "ff": sz["ff"]}} for i in range(sz["layers"])]}
+    for name, raw in (("bupozen", bup), ("rivudra", riv), ("buzarax", buz), ("naforax", naf), ("zuzezen", zuz), ("llama", llama)):
         if only and name not in only:
             continue
         ec = swiftllm_b200.EngineConfig(model_path="", use_dummy=False, block_size=16, gpu_mem_utilization=0.9, num_cpu_blocks=0,
                                         max_seqs_in_block_table=128, max_blocks_per_seq=512, max_batch_size=64,
                                         max_tokens_in_batch=16384, dtype=dtype)
         model = registry.create_model(ec, registry.model_config_from_dict(raw))
-        model.load_weights(synthetic_getter(seed=0, std=0.02, device="cuda", norm_offset=0.0 if name == "rivudra" else 1.0))   # Buzarax: scalar gains, depth weights and decays come from its loader's own synthetic rules
+        model.load_weights(synthetic_getter(seed=0, std=0.02, device="cuda", norm_offset=0.0 if name in ("rivudra", "zuzezen") else 1.0))   # Buzarax: scalar gains, depth weights and decays come from its loader's own synthetic rules
         model.init_kvcache_and_swap(64 * 4096 // 16 + 64)
         yield name, raw, model
         del model
@@ -224,7 +235,7 @@ def run_arch_compare(args):
             g = torch.Generator().manual_seed(0)
             prompts = [torch.randint(0, sz["vocab"], (prompt_len,), generator=g).tolist() for _ in range(n_prompts)]
             layers_pkg = "swiftllm_b200.worker.layers."
-            if name == "bupozen":
+            if name in ("bupozen", "zuzezen"):
                 mod, attrs = importlib.import_module(layers_pkg + "latent_attention"), ["latent_attention"]
             elif name in ("rivudra", "buzarax", "naforax"):
                 mod, attrs = importlib.import_module(layers_pkg + "window_attention"), ["window_attention"]
@@ -243,6 +254,12 @@ def run_arch_compare(args):
                          "input_conv": (importlib.import_module(layers_pkg + "sandwich_block"), "short_conv"),
                          "group_norms": (importlib.import_module(layers_pkg + "sandwich_block"), "group_norm_add_norm"),
                          "diff_combine": (importlib.import_module(layers_pkg + "window_attention"), "diff_combine")}
+            if name == "zuzezen":
+                extra = {"window_attention": (importlib.import_module(layers_pkg + "window_attention"), "window_attention"),
+                         "gated_linear_attention": (importlib.import_module(layers_pkg + "gated_linear_attention"), "gated_linear_attention"),
+                         "post_norms": (importlib.import_module(layers_pkg + "sequential_block"), "postnorm_add_mix"),
+                         "silu_glu": (importlib.import_module(layers_pkg + "feed_forward"), "silu_glu"),
+                         "sigmoid_gate": (importlib.import_module(layers_pkg + "latent_attention"), "sigmoid_gate_inplace")}
             extra_ms = {}
 
             def timed(fn, steps, warmup, after=None):
@@ -355,6 +372,36 @@ def run_arch_compare(args):
                     "group_norms": (nconv * ntok * Wd * 8, nconv * ntok * Wd * 14, nconv * dec_batch * Wd * 8, nconv * dec_batch * Wd * 14),
                     "diff_combine": (La * ntok * H * dv * 8, La * ntok * H * dv * 12, La * dec_batch * H * dv * 8, La * dec_batch * H * dv * 12),
                 }
+            elif name == "zuzezen":
+                # latent attention layers 0 and 3 of every four: full causal, q_lat + q_rot + out + the cache rows once (prefill), the
+                # cache rows (decode)
+                kinds = [i % 4 for i in range(L)]
+                Ll, Lw, Lg = sum(k in (0, 3) for k in kinds), kinds.count(1), kinds.count(2)
+                Lff = L - Lg
+                r, dr, Wn, D, nkv, Wd, F = 512, 64, sz["window"], sz["width"] // H, max(1, H // 4), sz["width"], sz["ff"]
+                ntok = n_prompts * prompt_len
+                fl_pre = Ll * n_prompts * (prompt_len * (prompt_len + 1) // 2) * H * (4 * r + 2 * dr)
+                by_pre = Ll * ntok * (r + dr + 2 * H * r + H * dr) * 2
+                fl_dec = Ll * dec_batch * (ctx + 1) * H * (4 * r + 2 * dr)
+                by_dec = Ll * dec_batch * (ctx + 1) * (r + dr) * 2
+                # label -> (prefill FLOPs, bytes, decode FLOPs, bytes).  Windowed attention: q + out + the key rows once (they are the
+                # values too), the visible rows (decode).  Gated linear attention: q, k, v, gate in and the product out (2 bytes), fp32
+                # decay logits, 4 dk dv FLOPs per token and head; decode reads and writes every sequence's fp32 state.  Post norms: the
+                # stream both ways, the sublayer's output in, the rounded stream out.
+                vis_pre = sum(min(p + 1, Wn + 4) for p in range(prompt_len)) * n_prompts
+                vis_dec = dec_batch * min(ctx + 1, Wn + 4)
+                gio = H * (3 * 128 * 2 + 128 * 4 + 2 * 128 * 2)
+                extra_roof = {
+                    "window_attention": (Lw * vis_pre * H * D * 4, Lw * ntok * (2 * H + nkv) * D * 2, Lw * vis_dec * H * D * 4,
+                                         Lw * vis_dec * nkv * (D * 2 + 4)),
+                    "gated_linear_attention": (Lg * ntok * H * 4 * 128 * 128, Lg * ntok * gio, Lg * dec_batch * H * 4 * 128 * 128,
+                                               Lg * dec_batch * (H * 128 * 128 * 8 + gio)),
+                    "post_norms": ((L + Lff) * ntok * Wd * 8, (L + Lff) * ntok * Wd * 12, (L + Lff) * dec_batch * Wd * 8,
+                                   (L + Lff) * dec_batch * Wd * 12),
+                    "silu_glu": (Lff * ntok * F * 8, Lff * ntok * F * 6, Lff * dec_batch * F * 8, Lff * dec_batch * F * 6),
+                    "sigmoid_gate": (Ll * ntok * H * 128 * 4, Ll * ntok * H * 128 * 6, Ll * dec_batch * H * 128 * 4,
+                                     Ll * dec_batch * H * 128 * 6),
+                }
             else:
                 D, nkv = sz["width"] // H, max(1, H // 4)
                 fl_pre = L * n_prompts * (prompt_len * (prompt_len + 1) // 2) * H * D * 4
@@ -366,7 +413,7 @@ def run_arch_compare(args):
                 t_min = max(fl / (peaks["bf16_tflops"] * 1e12), by / (peaks["hbm_gbs"] * 1e9)) * 1e3
                 return round(t_min / ms, 4) if ms > 0 else None
             other = {}
-            if name in ("buzarax", "naforax"):
+            if name in ("buzarax", "naforax", "zuzezen"):
                 for k, (fp, bp, fd, bd) in extra_roof.items():
                     other[k] = {"prefill_ms": round(pre_extra.get(k, 0.0), 3), "decode_ms": round(dec_extra.get(k, 0.0), 3),
                                 "prefill_roofline_frac": roof(fp, bp, pre_extra.get(k, 0.0)),

@@ -12,8 +12,9 @@ from oracle import bupozen as O
 from oracle import buzarax as _buzarax
 from oracle import naforax as _naforax
 from oracle import rivudra as _rivudra
+from oracle import zuzezen as _zuzezen
 
-_ORACLES = {"Bupozen": O, "Rivudra": _rivudra, "Buzarax": _buzarax, "Naforax": _naforax}
+_ORACLES = {"Bupozen": O, "Rivudra": _rivudra, "Buzarax": _buzarax, "Naforax": _naforax, "Zuzezen": _zuzezen}
 
 
 def oracle_of(cfg):

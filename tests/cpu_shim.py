@@ -192,14 +192,17 @@ def _latent_kv_store(dkv, norm_weight, cache, slot, block_table, st, r, dr, rot_
         cache[int(block_table[sq, p // bs]), slot, p % bs] = torch.cat([c[t], kr[t]])
 
 
-def _latent_attention(q_lat, q_rot, gate, cache, slot, block_table, st, out, rot_dims, window, scale, cos, sin):
+def _latent_attention(q_lat, q_rot, gate, cache, slot, block_table, st, out, rot_dims, window, scale, cos, sin, sink=None):
     r = q_lat.shape[2]
     qr = _rot_pairs(q_rot.float(), cos, sin, rot_dims)
     qa = torch.cat([q_lat.float(), qr], dim=-1) * scale                     # [T, H, r + dr]
     for t, (sq, p) in enumerate(zip(st.token_seq_ids.tolist(), st.token_positions.tolist())):
         lo = max(0, p - window + 1) if window > 0 else 0
         rows = _cache_rows(cache, slot, block_table, sq, list(range(lo, p + 1))).float()      # [n, r + dr]
-        pr = torch.softmax(qa[t] @ rows.T, dim=-1)                          # [H, n]
+        sc = qa[t] @ rows.T                                                 # [H, n]
+        if sink is not None:
+            sc = torch.cat([sc, sink[:, None]], dim=1)
+        pr = torch.softmax(sc, dim=-1)[:, :rows.shape[0]]
         o = pr @ rows[:, :r]
         if gate is not None:
             o = o * torch.sigmoid(gate[t].float())[:, None]
@@ -269,6 +272,16 @@ def _window_kv_store(k, v, cache, slot, block_table, st, kv_heads, dk, dv, rot_d
         cache[int(block_table[sq, p // bs]), slot, p % bs] = torch.cat([kr[t], v[t]])
 
 
+def _shared_kv_store(k, cache, slot, block_table, st, kv_heads, dk, eps):
+    T, bs, off = k.shape[0], cache.shape[2], (2 * kv_heads + 7) // 8 * 8
+    kf = k.float().view(T, kv_heads, dk)
+    inv = 1.0 / torch.sqrt((kf * kf).mean(-1) + eps)
+    for t, (sq, p) in enumerate(zip(st.token_seq_ids.tolist(), st.token_positions.tolist())):
+        row = cache[int(block_table[sq, p // bs]), slot, p % bs]
+        row[:off].view(torch.float32)[:kv_heads] = inv[t]
+        row[off:off + kv_heads * dk] = k[t]
+
+
 def _window_attention(q, gate, cache, slot, block_table, st, out, heads, kv_heads, dk, dv, rot_dims, window, scale, sink, cos, sin,
                       opt=None, vcos=None, vsin=None):
     T = q.shape[0]
@@ -286,12 +299,22 @@ def _window_attention(q, gate, cache, slot, block_table, st, out, heads, kv_head
         lo = max(0, p - window + 1) if window > 0 else 0
         if opt and opt.chunk > 0:
             lo = max(lo, p // opt.chunk * opt.chunk)
-        rows = _cache_rows(cache, slot, block_table, sq, list(range(lo, p + 1))).float()      # [n, G dk + G / vshare dv]
-        ks = rows[:, :kv_heads * dk].view(-1, kv_heads, dk).repeat_interleave(rep, dim=1)     # [n, H, dk]
-        vs = rows[:, kv_heads * dk:].view(-1, kv_heads // vshare, dv).repeat_interleave(rep * vshare, dim=1)
+        seen = list(range(min(opt.keep_first, lo) if opt and window > 0 else 0)) + list(range(lo, p + 1))
+        rows = _cache_rows(cache, slot, block_table, sq, seen)                                # [n, G dk + G / vshare dv]
+        if opt and opt.shared_kv:
+            off = (2 * kv_heads + 7) // 8 * 8
+            inv = rows[:, :off].contiguous().view(torch.float32)[:, :kv_heads]
+            vg = rows[:, off:off + kv_heads * dk].float().view(-1, kv_heads, dk)
+            ks, vs = ((vg * inv[:, :, None]).repeat_interleave(rep, dim=1), vg.repeat_interleave(rep, dim=1))
+        else:
+            rows = rows.float()
+            ks = rows[:, :kv_heads * dk].view(-1, kv_heads, dk).repeat_interleave(rep, dim=1)     # [n, H, dk]
+            vs = rows[:, kv_heads * dk:].view(-1, kv_heads // vshare, dv).repeat_interleave(rep * vshare, dim=1)
         sc = torch.einsum("hd,nhd->hn", qa[t], ks)
         if opt and opt.softcap > 0:
             sc = opt.softcap * torch.tanh(sc / opt.softcap)
+        if opt and opt.slopes is not None:
+            sc = sc - opt.slopes[:, None] * (p - torch.tensor(seen, dtype=torch.float32))[None, :]
         if sink:
             sc = torch.cat([sc, torch.zeros(heads, 1)], dim=1)
         pr = torch.softmax(sc, dim=-1)[:, :rows.shape[0]]
@@ -300,7 +323,8 @@ def _window_attention(q, gate, cache, slot, block_table, st, out, heads, kv_head
             o = _rot_any(o[None], vcos[t:t + 1], -vsin[t:t + 1], dv, halves)[0]
         o = o.reshape(heads * dv) * (opt.out_scale if opt else 1.0)
         if gate is not None:
-            o = o * torch.sigmoid(gate[t].float())
+            g = torch.sigmoid(gate[t].float())
+            o = o * (g.repeat_interleave(dv) if opt and opt.gate_per_head else g)
         out[t] = o.to(out.dtype)
 
 
@@ -430,8 +454,8 @@ def _segments(st):
     return [(sq, s[b], s[b + 1]) for b, sq in enumerate(st.seq_ids.tolist()) if s[b + 1] > s[b]]
 
 
-def _embed_pair_hash(tokens, st, last_token, embed, pairs, buckets, mul_prev, mul_cur, x_copy=None):
-    x = embed[tokens.long()].float()
+def _embed_pair_hash(tokens, st, last_token, embed, pairs, buckets, mul_prev, mul_cur, x_copy=None, scale=1.0):
+    x = embed[tokens.long()].float() * scale
     if pairs is not None:
         pos = st.token_positions.tolist()
         toks = tokens.tolist()
@@ -528,6 +552,32 @@ def _linear_attention(q, k, v, decay, state, st, heads, dk, dv):
     return out.reshape(T, heads * dv)
 
 
+def _gla(q, k, v, z, bias, tau, norm_w, eps, gate, state, st, heads, dk, dv):
+    T = q.shape[0]
+    qf, kf, vf = (q.float() * dk ** -0.5).view(T, heads, dk), k.float().view(T, heads, dk), v.float().view(T, heads, dv)
+    alpha = torch.exp(torch.nn.functional.logsigmoid(z + bias) / tau).view(T, heads, dk)
+    out = torch.zeros(T, heads, dv)
+    pos = st.token_positions.tolist()
+    for sq, lo, hi in _segments(st):
+        S = state[sq].clone() if pos[lo] > 0 else torch.zeros(heads, dk, dv)
+        for t in range(lo, hi):
+            S = alpha[t][:, :, None] * S + kf[t][:, :, None] * vf[t][:, None, :]
+            out[t] = torch.einsum("hkv,hk->hv", S, qf[t])
+        state[sq] = S
+    y = (_unit_rms(out, eps) * norm_w).reshape(T, heads * dv)
+    return (y * torch.nn.functional.silu(gate.float())).to(q.dtype)
+
+
+def _silu_glu(u):
+    F = u.shape[1] // 2
+    uf = u.float()
+    return (torch.nn.functional.silu(uf[:, :F]) * uf[:, F:]).to(u.dtype)
+
+
+def _sigmoid_gate_inplace(x, gate):
+    x.copy_((x.float() * torch.sigmoid(gate.float())).to(x.dtype))
+
+
 def _gated_rmsnorm(x, weight, gate, eps, out, out_scale=1.0):
     y = _unit_rms(x, eps) * weight * out_scale
     if gate is not None:
@@ -616,6 +666,14 @@ _PATCHES = [
     ("swiftllm_b200.worker.layers.linear_attention", "linear_attention", _linear_attention),
     ("swiftllm_b200.worker.layers.linear_attention", "gated_rmsnorm", _gated_rmsnorm),
     ("swiftllm_b200.worker.layers.window_attention", "diff_combine", _diff_combine),
+    ("swiftllm_b200.worker.layers.window_attention", "shared_kv_store", _shared_kv_store),
+    ("swiftllm_b200.worker.layers.latent_attention", "sigmoid_gate_inplace", _sigmoid_gate_inplace),
+    ("swiftllm_b200.worker.layers.gated_linear_attention", "gated_linear_attention", _gla),
+    ("swiftllm_b200.worker.layers.gated_linear_attention", "linear_f32_out", _linear_f32_out),
+    ("swiftllm_b200.worker.layers.feed_forward", "silu_glu", _silu_glu),
+    ("swiftllm_b200.worker.zuzezen_model", "embed_pair_hash", _embed_pair_hash),
+    ("swiftllm_b200.worker.zuzezen_model", "add_rmsnorm_f32", _add_rmsnorm_f32),
+    ("swiftllm_b200.worker.zuzezen_model", "linear_f32_out", _linear_f32_out),
     ("swiftllm_b200.worker.naforax_model", "embed_pair_hash", _embed_pair_hash),
     ("swiftllm_b200.worker.naforax_model", "tanh_cap_inplace", _tanh_cap_inplace),
     ("swiftllm_b200.worker.naforax_model", "group_norm_add_norm", _group_norm_add_norm),
