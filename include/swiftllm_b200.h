@@ -386,14 +386,15 @@ int sllm_gated_rmsnorm(const void* x, const void* weight, const void* gate, int6
 /* ---- Gated linear attention with per-sequence state (new, gla.cu); segments as for the recurrent mixers above.  Per head, with
  * alpha[t, d] = sigmoid(z[t, d] + bias[d])^inv_tau:  S <- diag(alpha) S + k v^T (dk x dv),  o = S^T (q * q_scale),
  * out[t] = o / sqrt(mean(o^2) + eps) * norm_w * silu(gate[t]).  q, k [T, heads * dk], v, gate, out [T, heads * dv] (dtype), z fp32
- * [T, heads * dk] (row strides in elements), bias fp32 [heads * dk], norm_w fp32 [dv], state fp32 [rows, heads, dk, dv],
- * o_workspace fp32 [T, heads * dv].  The first num_prefill_segs segments (num_prefill_tokens rows) are prompt portions, the rest
- * single decoded tokens: a hint for the launch shape, any split gives the same result up to rounding.  dk <= 512. */
+ * [T, heads * dk] (row strides in elements), bias fp32 [heads * dk], norm_w fp32 [dv], state fp32 [rows, heads, dk, dv].
+ * The first num_prefill_segs segments (num_prefill_tokens rows, the longest with max_prefill_len) are prompt portions, every other
+ * segment is ONE token.  workspace: fp32, at least gla_workspace_floats entries.  dk <= 512, dv <= 4096. */
+int64_t sllm_gla_workspace_floats(int64_t num_tokens, int num_prefill_segs, int64_t max_prefill_len, int num_heads, int dk, int dv);
 int sllm_gla(const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t v_stride, const void* z,
              int64_t z_stride, const void* bias, float inv_tau, float q_scale, const void* norm_w, float eps, const void* gate,
-             int64_t gate_stride, void* state, const void* seg_starts, const void* seq_ids, const void* tok_pos, void* o_workspace,
-             void* out, int64_t out_stride, int64_t num_tokens, int64_t num_prefill_tokens, int num_segs, int num_prefill_segs,
-             int num_heads, int dk, int dv, sllm_dtype_t dtype, sllm_stream_t stream);
+             int64_t gate_stride, void* state, const void* seg_starts, const void* seq_ids, const void* tok_pos, void* workspace,
+             int64_t workspace_floats, void* out, int64_t out_stride, int64_t num_tokens, int64_t num_prefill_tokens, int num_segs,
+             int num_prefill_segs, int64_t max_prefill_len, int num_heads, int dk, int dv, sllm_dtype_t dtype, sllm_stream_t stream);
 
 /* ---- Sandwich blocks: x <- x + mult * norm_b(sublayer(norm_a(x))) with RMS norms over `groups` equal consecutive parts of a row
  * (new, sandwich_ops.cu).  group_norm_add_norm: with y (dtype [T, width]) x (fp32, in place) += mult * y / rms_g(y) * wb; with

@@ -75,8 +75,9 @@ SIGNATURES = {
     "sllm_store_last_tokens": (_I, [_P, _P, _P, _P, _I, _P]),
     "sllm_silu_glu": (_I, [_P, _P, _L, _I, _I, _P]),
     "sllm_sigmoid_gate_inplace": (_I, [_P, _P, _L, _L, _I, _I, _P]),
-    "sllm_gla": (_I, [_P, _L, _P, _L, _P, _L, _P, _L, _P, _F, _F, _P, _F, _P, _L, _P, _P, _P, _P, _P, _P, _L, _L, _L, _I, _I, _I, _I,
-                      _I, _I, _P]),
+    "sllm_gla_workspace_floats": (_L, [_L, _I, _L, _I, _I, _I]),
+    "sllm_gla": (_I, [_P, _L, _P, _L, _P, _L, _P, _L, _P, _F, _F, _P, _F, _P, _L, _P, _P, _P, _P, _P, _L, _P, _L, _L, _L, _I, _I, _L,
+                      _I, _I, _I, _I, _P]),
     "sllm_postnorm_add_mix": (_I, [_P, _P, _P, _I, _F, _P, _I, _P, _P, _L, _I, _I, _P]),
     "sllm_tanh_cap_inplace": (_I, [_P, _L, _F, _I, _P]),
     "sllm_moe_route_sigmoid": (_I, [_P, _P, _P, _L, _I, _I, _P]),

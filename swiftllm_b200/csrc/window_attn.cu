@@ -299,9 +299,10 @@ __global__ void __launch_bounds__(WA_MAX_HPB * 32) window_attn_kernel(
 // reads then fall into eight different bank groups for every dk / dv.
 constexpr int WT_ROWS = 64;
 
+// EXT: the kernel knows slopes, kept first positions, gates per head and shared_kv rows (compiled out otherwise).
 // WT_KEYS: keys per tile (32 or 64).  Smaller tiles leave room for more CTAs per SM (prompt portions: many CTAs, latency-bound);
 // larger ones keep more bytes in flight per CTA (decoded tokens: few CTAs that walk their window alone).
-template <typename T, int DMAX, int WT_KEYS>
+template <typename T, int DMAX, int WT_KEYS, bool EXT>
 __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_kernel(
     const T* __restrict__ q, int64_t q_stride_t, const float* __restrict__ cosb, const float* __restrict__ sinb,
     const T* __restrict__ gate, int64_t gate_stride_t, const T* __restrict__ cache, int n_slots, int slot, int block_size,
@@ -309,8 +310,11 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
     const int* __restrict__ tok_pos, T* __restrict__ out, int64_t out_stride_t, int row0, int nrows, int qt, int hq, int hqp_log2,
     int H, int G, int dk, int dv, int rot_dims, int window, float scale_log2, float sink, int halves, float qk_norm_eps,
     float softcap, const float* __restrict__ vcos, const float* __restrict__ vsin, float out_scale,
-    const float* __restrict__ qnorm_w, float prenorm_eps, int chunk, int vshare, int out_f32, const float* __restrict__ slopes,
-    int keep_first, int gate_per_head, int shared_kv) {
+    const float* __restrict__ qnorm_w, float prenorm_eps, int chunk, int vshare, int out_f32, const float* __restrict__ slopes_,
+    int keep_first_, int gate_per_head_, int shared_kv_) {
+    const float* slopes = EXT ? slopes_ : nullptr;
+    const int keep_first = EXT ? keep_first_ : 0;
+    const bool gate_per_head = EXT && gate_per_head_, shared_kv = EXT && shared_kv_;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int PQ = dk * 2 + 16, PK = dk * 2 + 16, PV = dv * 2 + 16;            // row pitches in bytes
     unsigned char* Qs = smem_raw;                                              // [64][PQ]
@@ -597,6 +601,264 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
     }
 }
 
+// ------------------------------------------------------------------ attention of single decoded tokens (tensor cores, 16-bit storage)
+// One CTA = one token and key/value group; its (at most 16) query heads are the M dimension of the MMA tiles.  The token's visible
+// keys are split over the CTA's four WARPS: warp w walks the tiles w, w + 4, .. of KT keys through a two-stage cp.async ring of its
+// own (no CTA barrier inside the loop) with its own running (maximum, sum, output); the four results are merged through shared memory
+// at the end.  Queries are held in registers as MMA fragments for the whole walk.  Same options as the kernel above.
+constexpr int WD_WARPS = 4;
+
+template <typename T, int DMAX, int KT, bool EXT>
+__global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(
+    const T* __restrict__ q, int64_t q_stride_t, const float* __restrict__ cosb, const float* __restrict__ sinb,
+    const T* __restrict__ gate, int64_t gate_stride_t, const T* __restrict__ cache, int n_slots, int slot, int block_size,
+    const int* __restrict__ block_table, int max_blocks_per_seq, const int* __restrict__ tok_seq,
+    const int* __restrict__ tok_pos, T* __restrict__ out, int64_t out_stride_t, int row0, int hq,
+    int G, int dk, int dv, int rot_dims, int window, float scale_log2, float sink, int halves, float qk_norm_eps,
+    float softcap, const float* __restrict__ vcos, const float* __restrict__ vsin, float out_scale,
+    const float* __restrict__ qnorm_w, float prenorm_eps, int chunk, int vshare, int out_f32, const float* __restrict__ slopes_,
+    int keep_first_, int gate_per_head_, int shared_kv_) {
+    const float* slopes = EXT ? slopes_ : nullptr;
+    const int keep_first = EXT ? keep_first_ : 0;
+    const bool gate_per_head = EXT && gate_per_head_, shared_kv = EXT && shared_kv_;
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    const int PQ = dk * 2 + 16, PK = dk * 2 + 16, PV = dv * 2 + 16;            // row pitches in bytes
+    const int stage_bytes = KT * (PK + (shared_kv ? (int)sizeof(float) : PV));
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    unsigned char* Qs = smem_raw;                                              // [16][PQ]
+    unsigned char* Ws = Qs + 16 * PQ + warp * 2 * stage_bytes;                 // this warp's two stages: K [KT][PK], V [KT][PV] | 1 / rms [KT]
+    const int g = blockIdx.y;
+    const int64_t t = row0 + blockIdx.x;
+    const int pos = tok_pos[t];
+    const int* bt = block_table + (int64_t)tok_seq[t] * max_blocks_per_seq;
+    const int row_elems = shared_kv ? shared_kv_row(G, dk) : G * dk + (G / vshare) * dv;
+    const int koff = (shared_kv ? shared_kv_key_offset(G) : 0) + g * dk, voff = G * dk + (g / vshare) * dv;
+    const int ck = dk >> 3, cv = shared_kv ? 0 : dv >> 3;                      // 16-byte chunks per key / value row
+    int lprk = 1, lprv = 1;                                                    // lanes per row: the largest power of two <= chunks
+    while (lprk * 2 <= ck && lprk < 32) lprk *= 2;
+    while (lprv * 2 <= cv && lprv < 32) lprv *= 2;
+    int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    if (chunk > 0) lo = max(lo, pos / chunk * chunk);
+    const int nk = window > 0 ? min(keep_first, lo) : 0;
+    const int total = nk + pos - lo + 1;
+    const int ntiles = (total - 1) / KT + 1;
+
+    auto load_tile = [&](int it, int st) {
+        unsigned char* K = Ws + st * stage_bytes;
+        unsigned char* V = K + KT * PK;
+        // lane l < KT finds row l of the tile; the copies then take whole rows with neighbouring lanes
+        const int e = it * KT + lane;
+        const bool ok = lane < KT && e < total;
+        long long row = 0;
+        if (ok) {
+            const int kp = key_position(e, nk, lo), b = kp / block_size;
+            row = (((long long)bt[b] * n_slots + slot) * block_size + (kp - b * block_size)) * row_elems;
+        }
+        if (shared_kv && lane < KT) {
+            float* ki = reinterpret_cast<float*>(V) + lane;
+            if (ok) cp_async4(smem_u32(ki), cache + row + 2 * g);
+            else *ki = 0.f;
+        }
+        const unsigned live = __ballot_sync(0xffffffffu, ok);
+        for (int r0 = 0; r0 < KT; r0 += 32 / lprk) {
+            const int r = r0 + lane / lprk;
+            const long long base = __shfl_sync(0xffffffffu, row, r & 31);
+            const int nb = (live >> (r & 31)) & 1 ? 16 : 0;
+            if (r < KT)
+                for (int ch = lane % lprk; ch < ck; ch += lprk) cp_async16(smem_u32(K + r * PK + ch * 16), cache + base + (nb ? koff + ch * 8 : 0), nb);
+        }
+        if (!shared_kv)
+            for (int r0 = 0; r0 < KT; r0 += 32 / lprv) {
+                const int r = r0 + lane / lprv;
+                const long long base = __shfl_sync(0xffffffffu, row, r & 31);
+                const int nb = (live >> (r & 31)) & 1 ? 16 : 0;
+                if (r < KT)
+                    for (int ch = lane % lprv; ch < cv; ch += lprv) cp_async16(smem_u32(V + r * PV + ch * 16), cache + base + (nb ? voff + ch * 8 : 0), nb);
+            }
+        cp_async_commit();
+    };
+    if (warp < ntiles) load_tile(warp, 0);
+
+    // ---- queries: rows past the group's heads are zeros; eight threads per row
+    {
+        const int r = tid >> 3, part = tid & 7;
+        const bool live = r < hq;
+        const int half = rot_dims >> 1;
+        const T* qr = q + t * q_stride_t + (int64_t)(g * hq + (live ? r : 0)) * dk;
+        const float* cs = cosb != nullptr ? cosb + t * half : nullptr;
+        const float* sn = sinb != nullptr ? sinb + t * half : nullptr;
+        float pinv = 1.f;
+        if (qnorm_w != nullptr) {
+            float s0 = 0.f;
+            for (int i = part; i < dk; i += 8) { const float a = ldf(qr + i); s0 += a * a; }
+            s0 += __shfl_xor_sync(0xffffffffu, s0, 1); s0 += __shfl_xor_sync(0xffffffffu, s0, 2); s0 += __shfl_xor_sync(0xffffffffu, s0, 4);
+            pinv = 1.f / sqrtf(s0 / (float)dk + prenorm_eps);
+        }
+        float inv = 1.f;
+        if (qk_norm_eps >= 0.f) {
+            float ss = 0.f;
+            for (int i = part; i < dk; i += 8) { const float a = rot_entry(qr, i, rot_dims, halves, cs, sn, pinv, qnorm_w); ss += a * a; }
+            ss += __shfl_xor_sync(0xffffffffu, ss, 1); ss += __shfl_xor_sync(0xffffffffu, ss, 2); ss += __shfl_xor_sync(0xffffffffu, ss, 4);
+            inv = 1.f / sqrtf(ss / (float)dk + qk_norm_eps);
+        }
+        for (int i = part; i < (dk >> 1); i += 8) {
+            float a = 0.f, b = 0.f;
+            if (live) {
+                a = rot_entry(qr, 2 * i, rot_dims, halves, cs, sn, pinv, qnorm_w) * inv;
+                b = rot_entry(qr, 2 * i + 1, rot_dims, halves, cs, sn, pinv, qnorm_w) * inv;
+            }
+            *reinterpret_cast<uint32_t*>(Qs + r * PQ + i * 4) = pack2<T>(a, b);
+        }
+    }
+    __syncthreads();
+    uint32_t qf[DMAX / 16][4];
+#pragma unroll
+    for (int kk = 0; kk < DMAX / 16; kk++)
+        if (kk * 16 < dk)
+            ldmatrix_x4(smem_u32(Qs + ((lane & 7) + ((lane >> 3) & 1) * 8) * PQ + (kk * 16 + (lane >> 4) * 8) * 2), qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3]);
+
+    const int r_a = lane >> 2, r_b = r_a + 8;
+    const float cap_in = softcap > 0.f ? scale_log2 * 0.6931471805599453f / softcap : 0.f;
+    const float cap_out = softcap * 1.4426950408889634f;
+    const float sl_a = slopes != nullptr && r_a < hq ? slopes[g * hq + r_a] * 1.4426950408889634f : 0.f;
+    const float sl_b = slopes != nullptr && r_b < hq ? slopes[g * hq + r_b] * 1.4426950408889634f : 0.f;
+    float m_a = sink > 0.f && warp == 0 ? 0.f : -INFINITY, m_b = m_a;
+    float l_a = (lane & 3) == 0 && warp == 0 ? sink : 0.f, l_b = l_a;
+    float o[DMAX / 8][4];
+#pragma unroll
+    for (int nt = 0; nt < DMAX / 8; nt++) { o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f; }
+
+    int st = 0;
+    for (int it = warp; it < ntiles; it += WD_WARPS, st ^= 1) {
+        if (it + WD_WARPS < ntiles) { load_tile(it + WD_WARPS, st ^ 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
+        __syncwarp();                                                          // the tile is visible to the whole warp
+        const unsigned char* Kt = Ws + st * stage_bytes;
+        const unsigned char* Vt = shared_kv ? Kt : Kt + KT * PK;
+        const int PVt = shared_kv ? PK : PV;
+        float sc[KT / 8][4];
+#pragma unroll
+        for (int nt = 0; nt < KT / 8; nt++) { sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f; }
+#pragma unroll
+        for (int kk = 0; kk < DMAX / 16; kk++) {
+            if (kk * 16 < dk) {
+#pragma unroll
+                for (int np = 0; np < KT / 16; np++) {
+                    uint32_t b0, b1, b2, b3;
+                    ldmatrix_x4(smem_u32(Kt + (np * 16 + (lane >> 4) * 8 + (lane & 7)) * PK + (kk * 16 + ((lane >> 3) & 1) * 8) * 2), b0, b1, b2, b3);
+                    mma_16816<T>(sc[2 * np], qf[kk], b0, b1);
+                    mma_16816<T>(sc[2 * np + 1], qf[kk], b2, b3);
+                }
+            }
+        }
+        const float* ki = reinterpret_cast<const float*>(Kt + KT * PK) + (lane & 3) * 2;
+        float mx_a = -INFINITY, mx_b = -INFINITY;
+#pragma unroll
+        for (int nt = 0; nt < KT / 8; nt++) {
+            if (shared_kv) {
+                const float2 f = *reinterpret_cast<const float2*>(ki + nt * 8);
+                sc[nt][0] *= f.x; sc[nt][1] *= f.y; sc[nt][2] *= f.x; sc[nt][3] *= f.y;
+            }
+#pragma unroll
+            for (int e = 0; e < 2; e++) {
+                const int v = it * KT + nt * 8 + (lane & 3) * 2 + e;           // every entry of the list below `total` is visible
+                float sa = softcap > 0.f ? cap_out * tanhf(sc[nt][e] * cap_in) : sc[nt][e] * scale_log2;
+                float sb = softcap > 0.f ? cap_out * tanhf(sc[nt][2 + e] * cap_in) : sc[nt][2 + e] * scale_log2;
+                if (EXT) {
+                    const float dist = (float)(pos - key_position(v, nk, lo));
+                    sa -= sl_a * dist;
+                    sb -= sl_b * dist;
+                }
+                sc[nt][e] = v < total ? sa : -INFINITY;
+                sc[nt][2 + e] = v < total ? sb : -INFINITY;
+                mx_a = fmaxf(mx_a, sc[nt][e]);
+                mx_b = fmaxf(mx_b, sc[nt][2 + e]);
+            }
+        }
+        mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 1)); mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 2));
+        mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 1)); mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 2));
+        const float mn_a = fmaxf(m_a, mx_a), mn_b = fmaxf(m_b, mx_b);          // finite: a tile has at least one visible key
+        const float al_a = exp2f(m_a - mn_a), al_b = exp2f(m_b - mn_b);
+        m_a = mn_a; m_b = mn_b;
+        l_a *= al_a; l_b *= al_b;
+#pragma unroll
+        for (int nt = 0; nt < DMAX / 8; nt++) { o[nt][0] *= al_a; o[nt][1] *= al_a; o[nt][2] *= al_b; o[nt][3] *= al_b; }
+        uint32_t pa[KT / 16][4];
+#pragma unroll
+        for (int nt = 0; nt < KT / 8; nt++) {
+            const float p0 = exp2f(sc[nt][0] - mn_a), p1 = exp2f(sc[nt][1] - mn_a);
+            const float p2 = exp2f(sc[nt][2] - mn_b), p3 = exp2f(sc[nt][3] - mn_b);
+            l_a += p0 + p1; l_b += p2 + p3;
+            pa[nt >> 1][(nt & 1) * 2] = pack2<T>(p0, p1);
+            pa[nt >> 1][(nt & 1) * 2 + 1] = pack2<T>(p2, p3);
+        }
+#pragma unroll
+        for (int kk = 0; kk < KT / 16; kk++) {
+#pragma unroll
+            for (int np = 0; np < DMAX / 16; np++) {
+                if (np * 16 < dv) {
+                    uint32_t b0, b1, b2, b3;
+                    ldmatrix_x4_trans(smem_u32(Vt + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PVt + (np * 16 + (lane >> 4) * 8) * 2), b0, b1, b2, b3);
+                    mma_16816<T>(o[2 * np], pa[kk], b0, b1);
+                    mma_16816<T>(o[2 * np + 1], pa[kk], b2, b3);
+                }
+            }
+        }
+        __syncwarp();                                                          // the stage may be overwritten
+    }
+
+    // ---- merge the warps, (turn back,) gate, store
+    l_a += __shfl_xor_sync(0xffffffffu, l_a, 1); l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
+    l_b += __shfl_xor_sync(0xffffffffu, l_b, 1); l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
+    __syncthreads();                                                           // every warp is done with its tiles
+    float* Om = reinterpret_cast<float*>(smem_raw);                            // [WD_WARPS][hq][dv]
+    float* Ms = Om + WD_WARPS * hq * dv;                                       // [WD_WARPS][16] maximum, then [WD_WARPS][16] sum
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+        const int r = e ? r_b : r_a;
+        if (r >= hq) continue;
+        if ((lane & 3) == 0) { Ms[warp * 16 + r] = e ? m_b : m_a; Ms[(WD_WARPS + warp) * 16 + r] = e ? l_b : l_a; }
+#pragma unroll
+        for (int nt = 0; nt < DMAX / 8; nt++) {
+            const int d = nt * 8 + (lane & 3) * 2;
+            if (d < dv) *reinterpret_cast<float2*>(Om + (warp * hq + r) * dv + d) = make_float2(o[nt][2 * e], o[nt][2 * e + 1]);
+        }
+    }
+    __syncthreads();
+    const int n_out = hq * dv;
+    for (int i = tid; i < n_out; i += WD_WARPS * 32) {                         // slot 0 <- the normalised output
+        const int r = i / dv;
+        float M = Ms[r];
+#pragma unroll
+        for (int w = 1; w < WD_WARPS; w++) M = fmaxf(M, Ms[w * 16 + r]);
+        float L = 0.f, y = 0.f;
+#pragma unroll
+        for (int w = 0; w < WD_WARPS; w++) {
+            const float f = exp2f(Ms[w * 16 + r] - M);                         // 0 for a warp that saw no key
+            L += f * Ms[(WD_WARPS + w) * 16 + r];
+            y += f * Om[w * n_out + i];
+        }
+        Om[i] = y / L;
+    }
+    if (vcos != nullptr) __syncthreads();                                      // the turn back reads a neighbour's entry
+    const int hv = dv >> 1;
+    for (int i = tid; i < n_out; i += WD_WARPS * 32) {
+        const int r = i / dv, d = i - r * dv;
+        float y = Om[i];
+        if (vcos != nullptr) {
+            int m, second;
+            if (halves) { second = d >= hv; m = second ? d - hv : d; } else { second = d & 1; m = d >> 1; }
+            const float a = Om[r * dv + (halves ? m : 2 * m)], b = Om[r * dv + (halves ? m + hv : 2 * m + 1)];
+            const float c = vcos[t * hv + m], sn = vsin[t * hv + m];
+            y = second ? b * c - a * sn : a * c + b * sn;
+        }
+        y *= out_scale;
+        const int64_t h = g * hq + r;
+        if (gate != nullptr) y *= 1.f / (1.f + __expf(-ldf(gate + t * gate_stride_t + (gate_per_head ? h : h * dv + d))));
+        if (out_f32) reinterpret_cast<float*>(out)[t * out_stride_t + h * dv + d] = y;
+        else stf(out + t * out_stride_t + h * dv + d, y);
+    }
+}
+
 // ------------------------------------------------------------------ two maps -> one head
 // a: fp32 [T, G, 2, hq, dv] (the attention above with vshare = 2 and queries ordered [key/value head][map][head of the group]).
 // One warp per (token, head h = g hq + hh): o = a[g, 0, hh] - lambda a[g, 1, hh]; out = o / sqrt(mean(o^2) + eps) * factor *
@@ -637,7 +899,7 @@ __global__ void __launch_bounds__(256) diff_combine_kernel(const float* __restri
 static bool g_window_simt = false;
 
 // rows [0, num_prefill) are prompt portions (many consecutive tokens of a sequence share a CTA), the rest single decoded tokens
-template <typename T, int DMAX>
+template <typename T, int DMAX, bool EXT>
 static int launch_window_attn_mma(const void* q, int64_t q_stride_t, const void* cosb, const void* sinb, const void* gate,
                                   int64_t gate_stride_t, const void* cache, int n_slots, int slot, int block_size,
                                   const void* block_table, int max_blocks_per_seq, const void* tok_seq, const void* tok_pos,
@@ -650,9 +912,13 @@ static int launch_window_attn_mma(const void* q, int64_t q_stride_t, const void*
     const int hq = H / G;
     int hqp_log2 = 0;
     while ((1 << hqp_log2) < hq) hqp_log2++;
-    auto kern_prompt = window_attn_mma_kernel<T, DMAX, 32>;
-    auto kern_decode = window_attn_mma_kernel<T, DMAX, 64>;
+    auto kern_prompt = window_attn_mma_kernel<T, DMAX, 32, EXT>;
+    auto kern_decode = window_attn_mma_kernel<T, DMAX, 64, EXT>;
+    // single decoded tokens of up to 16 heads per group: keys split over the warps of a CTA; small tiles where a row is long
+    constexpr int KT = DMAX == 64 || EXT ? 32 : 16;
+    auto kern_split = window_attn_decode_kernel<T, DMAX, KT, EXT>;
     if (first_use_on_this_device(attr_mask)) {
+        cudaFuncSetAttribute(kern_split, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
         cudaFuncSetAttribute(kern_prompt, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);
         cudaFuncSetAttribute(kern_decode, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);
     }
@@ -663,6 +929,18 @@ static int launch_window_attn_mma(const void* q, int64_t q_stride_t, const void*
     for (int k = 0; k < 2; k++) {
         const int64_t first = parts[k][0], count = parts[k][1];
         if (count <= 0) continue;
+        if (k == 1 && hq <= 16) {
+            size_t smem = 16 * (size_t)(dk * 2 + 16) + WD_WARPS * 2 * (size_t)KT * ((dk * 2 + 16) + (shared_kv ? sizeof(float) : dv * 2 + 16));
+            const size_t merge = ((size_t)WD_WARPS * hq * dv + 2 * WD_WARPS * 16) * sizeof(float);
+            if (smem < merge) smem = merge;
+            kern_split<<<dim3((unsigned)count, (unsigned)G), WD_WARPS * 32, smem, stream>>>(
+                (const T*)q, q_stride_t, (const float*)cosb, (const float*)sinb, (const T*)gate, gate_stride_t, (const T*)cache,
+                n_slots, slot, block_size, (const int*)block_table, max_blocks_per_seq, (const int*)tok_seq, (const int*)tok_pos,
+                (T*)out, out_stride_t, (int)first, hq, G, dk, dv, rot_dims, window, scale_log2, sink, halves, qk_norm_eps, softcap,
+                (const float*)vcos, (const float*)vsin, out_scale, (const float*)qnorm_w, prenorm_eps, chunk, vshare, out_f32,
+                (const float*)slopes, keep_first, gate_per_head, shared_kv);
+            continue;
+        }
         const int qt = k == 0 ? WT_ROWS >> hqp_log2 : 1;
         // measured on B200 (128 + 128 per head): prompt portions 24 - 26 % faster with 32-key tiles (three CTAs per SM instead of
         // two); decoded tokens faster with 64-key tiles at 512 CTAs (357 vs 385 us), with 32-key tiles at 2048 CTAs (950 vs 1220 us)
@@ -789,14 +1067,17 @@ int sllm_window_attention(const void* q, int64_t q_stride_t, const void* cosb, c
     const int hq = num_heads / num_kv_heads;
     if (!g_window_simt && dtype != SLLM_F32 && dk % 16 == 0 && dv % 16 == 0 && dk <= 128 && dv <= 128 && hq <= WT_ROWS &&
         num_tokens < (1ll << 31)) {
-#define WA_MMA(DMAX)                                                                                                        \
-    SLLM_DISPATCH_DTYPE(dtype, return (launch_window_attn_mma<T, DMAX>(q, q_stride_t, cosb, sinb, gate, gate_stride_t, cache,  \
+#define WA_MMA(DMAX, EXT)                                                                                                        \
+    SLLM_DISPATCH_DTYPE(dtype, return (launch_window_attn_mma<T, DMAX, EXT>(q, q_stride_t, cosb, sinb, gate, gate_stride_t, cache,  \
         n_slots, slot, block_size, block_table, max_blocks_per_seq, tok_seq, tok_pos, out, out_stride_t, num_tokens,         \
         num_prefill_tokens, num_heads, num_kv_heads, dk, dv, rot_dims, window, scale, sinkw, pair_halves, qk_norm_eps, softcap, \
         vcos, vsin, out_scale, qnorm_w, prenorm_eps, chunk, vshare, out_f32, slopes, keep_first, gate_per_head, shared_kv,        \
         (cudaStream_t)stream)))
-        if (dk <= 64 && dv <= 64) { WA_MMA(64); }
-        else { WA_MMA(128); }
+        const bool ext = slopes != nullptr || keep_first > 0 || gate_per_head || shared_kv;
+        const bool small = dk <= 64 && dv <= 64;
+        if (ext) { if (small) { WA_MMA(64, true); } else { WA_MMA(128, true); } }
+        else if (small) { WA_MMA(64, false); }
+        else { WA_MMA(128, false); }
 #undef WA_MMA
     }
 #define WA_LAUNCH(KR)                                                                                                      \

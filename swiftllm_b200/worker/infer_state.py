@@ -68,5 +68,6 @@ class TokenInferState:
     ignore_kvcache: bool = False                    # memory-profiling forward: no cache store, no attention
     # rotary angle tables of the step, keyed by (base, dims[, scaling]): (cos, sin) fp32 [num_tokens, dims / 2]
     rotary: dict = dataclasses.field(default_factory=dict)
+    max_prefill_len: int = 0                        # tokens of the step's longest prompt portion
     # [batch_size + 1] first row of every sequence of the step, closed with num_tokens (kernels that walk a sequence's rows)
     seg_starts: Optional[torch.Tensor] = None

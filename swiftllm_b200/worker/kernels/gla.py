@@ -23,13 +23,14 @@ def gated_linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z:
     assert bias.shape == (heads * dk,) and norm_w.shape == (dv,) and state.is_contiguous() and state.shape[1:] == (heads, dk, dv)
     _lib.require_device(q)
     st = infer_state
-    ws = torch.empty((T, heads * dv), dtype=torch.float32, device=q.device)
     out = torch.empty((T, heads * dv), dtype=q.dtype, device=q.device)
-    nseg = min(st.batch_size, max(0, int(getattr(st, "num_prefill_seqs", st.batch_size))))
-    npre = min(T, max(0, int(getattr(st, "num_prefill_tokens", T))))
+    nseg, npre = st.num_prefill_seqs, st.num_prefill_tokens
+    longest = min(npre, st.max_prefill_len)
+    size = _lib.lib().sllm_gla_workspace_floats(T, nseg, longest, heads, dk, dv)
+    ws = torch.empty((size,), dtype=torch.float32, device=q.device)
     _lib.check(_lib.lib().sllm_gla(
         q.data_ptr(), _stride0(q), k.data_ptr(), _stride0(k), v.data_ptr(), _stride0(v), z.data_ptr(), _stride0(z), bias.data_ptr(),
         1.0 / tau, dk ** -0.5, norm_w.data_ptr(), eps, gate.data_ptr(), _stride0(gate), state.data_ptr(), st.seg_starts.data_ptr(),
-        st.seq_ids.data_ptr(), st.token_positions.data_ptr(), ws.data_ptr(), out.data_ptr(), heads * dv, T, npre, st.batch_size, nseg,
-        heads, dk, dv, _lib.dtype_tag_f32(q.dtype), _lib.stream()), "gla")
+        st.seq_ids.data_ptr(), st.token_positions.data_ptr(), ws.data_ptr(), size, out.data_ptr(), heads * dv, T, npre, st.batch_size,
+        nseg, longest, heads, dk, dv, _lib.dtype_tag_f32(q.dtype), _lib.stream()), "gla")
     return out

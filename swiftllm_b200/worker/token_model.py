@@ -218,7 +218,7 @@ class TokenBatchModel(PagedModelBase):
             batch_size=batch_size, num_tokens=num_tokens, seq_ids=seq_ids, num_prefill_seqs=num_prefill_seqs,
             num_decoding_seqs=batch_size - num_prefill_seqs, num_prefill_tokens=num_prefill_tokens, token_seq_ids=t_seq,
             token_positions=t_pos, output_rows=rows, ignore_kvcache=ignore_kvcache, rotary=self._rotary_tables(t_pos),
-            seg_starts=seg)
+            max_prefill_len=max(prefill_lens, default=0), seg_starts=seg)
         logits = self._forward(ids, st)
         self.last_logits = logits[batch_size:].float() if logit_rows else None
         return torch.argmax(logits[:batch_size], dim=1)
