@@ -344,7 +344,7 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
         int lo = (window > 0 && pos0 - window + 1 > 0) ? pos0 - window + 1 : 0;
         if (chunk > 0) lo = max(lo, pos0 / chunk * chunk);
         const int hi = pos0 + n - 1;
-        const int nk = window > 0 ? min(keep_first, lo) : 0;
+        const int nk = EXT && window > 0 ? min(keep_first, lo) : 0;
         const int total = nk + hi - lo + 1;                                    // keys the segment's rows see together
         const int ntiles = (total - 1) / WT_KEYS + 1;
         __syncthreads();                                                       // the previous segment's tiles and queries are done with
@@ -444,7 +444,7 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
             __syncthreads();                                                   // tile `it` (and, first time, the queries) visible
             const int base = it * WT_KEYS;                                     // the tile's first entry in the list of visible keys
             const int kp_first = key_position(base, nk, lo), kp_last = key_position(base + WT_KEYS - 1, nk, lo);
-            if (warp_live && kp_first <= w_hi && (kp_last >= w_lo || kp_first < keep_first)) {
+            if (warp_live && kp_first <= w_hi && (kp_last >= w_lo || (EXT && kp_first < keep_first))) {
                 const unsigned char* Kt = Ks + (it & 1) * WT_KEYS * PK;
                 const unsigned char* Vt = Vs + (it & 1) * WT_KEYS * PV;
                 float sc[WT_KEYS / 8][4];
@@ -481,12 +481,14 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
 #pragma unroll
                     for (int e = 0; e < 2; e++) {
                         const int kp = key_position(base + nt * 8 + (lane & 3) * 2 + e, nk, lo);
-                        const bool kept = kp < keep_first;
+                        const bool kept = EXT && kp < keep_first;
                         const bool va = live_a && kp <= pos_a && (kp >= lo_a || kept), vb = live_b && kp <= pos_b && (kp >= lo_b || kept);
                         float sa = softcap > 0.f ? cap_out * tanhf(sc[nt][e] * cap_in) : sc[nt][e] * scale_log2;
                         float sb = softcap > 0.f ? cap_out * tanhf(sc[nt][2 + e] * cap_in) : sc[nt][2 + e] * scale_log2;
-                        sa -= sl_a * (float)(pos_a - kp);
-                        sb -= sl_b * (float)(pos_b - kp);
+                        if (EXT) {
+                            sa -= sl_a * (float)(pos_a - kp);
+                            sb -= sl_b * (float)(pos_b - kp);
+                        }
                         sc[nt][e] = va ? sa : -INFINITY;
                         sc[nt][2 + e] = vb ? sb : -INFINITY;
                         mx_a = fmaxf(mx_a, sc[nt][e]);
@@ -602,13 +604,22 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
 }
 
 // ------------------------------------------------------------------ attention of single decoded tokens (tensor cores, 16-bit storage)
-// One CTA = one token and key/value group; its (at most 16) query heads are the M dimension of the MMA tiles.  The token's visible
-// keys are split over the CTA's four WARPS: warp w walks the tiles w, w + 4, .. of KT keys through a two-stage cp.async ring of its
-// own (no CTA barrier inside the loop) with its own running (maximum, sum, output); the four results are merged through shared memory
-// at the end.  Queries are held in registers as MMA fragments for the whole walk.  Same options as the kernel above.
+// One CTA = one token and key/value group of at most 8 NH query heads.  The token's visible keys are split over the CTA's four WARPS:
+// warp w walks the tiles w, w + 4, .. of KT keys through a cp.async ring of its own (no CTA barrier inside the loop) with its own
+// running (maximum, sum, output); the four results are merged through shared memory at the end.  The products are taken transposed, so
+// that the few heads are the narrow side of the MMA tiles: S^T [keys, heads] = K Q^T with Q^T in registers for the whole walk, then
+// O^T [dv, heads] += V^T P^T, where P^T is S^T's fragment turned by movmatrix.  Same options as the kernel above.
 constexpr int WD_WARPS = 4;
+constexpr int WD_STAGES = 3;
 
-template <typename T, int DMAX, int KT, bool EXT>
+// the 8 x 8 matrix of 16-bit entries held by the warp, transposed
+__device__ __forceinline__ uint32_t movmatrix_trans(uint32_t x) {
+    uint32_t y;
+    asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(y) : "r"(x));
+    return y;
+}
+
+template <typename T, int DMAX, int KT, int NH, bool EXT>
 __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(
     const T* __restrict__ q, int64_t q_stride_t, const float* __restrict__ cosb, const float* __restrict__ sinb,
     const T* __restrict__ gate, int64_t gate_stride_t, const T* __restrict__ cache, int n_slots, int slot, int block_size,
@@ -626,58 +637,55 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(
     const int stage_bytes = KT * (PK + (shared_kv ? (int)sizeof(float) : PV));
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     unsigned char* Qs = smem_raw;                                              // [16][PQ]
-    unsigned char* Ws = Qs + 16 * PQ + warp * 2 * stage_bytes;                 // this warp's two stages: K [KT][PK], V [KT][PV] | 1 / rms [KT]
+    unsigned char* Ws = Qs + 16 * PQ + warp * WD_STAGES * stage_bytes;         // this warp's stages: K [KT][PK], V [KT][PV] | 1 / rms [KT]
+    const uint32_t ws_a = smem_u32(Ws);
     const int g = blockIdx.y;
     const int64_t t = row0 + blockIdx.x;
     const int pos = tok_pos[t];
     const int* bt = block_table + (int64_t)tok_seq[t] * max_blocks_per_seq;
     const int row_elems = shared_kv ? shared_kv_row(G, dk) : G * dk + (G / vshare) * dv;
-    const int koff = (shared_kv ? shared_kv_key_offset(G) : 0) + g * dk, voff = G * dk + (g / vshare) * dv;
-    const int ck = dk >> 3, cv = shared_kv ? 0 : dv >> 3;                      // 16-byte chunks per key / value row
-    int lprk = 1, lprv = 1;                                                    // lanes per row: the largest power of two <= chunks
-    while (lprk * 2 <= ck && lprk < 32) lprk *= 2;
-    while (lprv * 2 <= cv && lprv < 32) lprv *= 2;
     int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
     if (chunk > 0) lo = max(lo, pos / chunk * chunk);
-    const int nk = window > 0 ? min(keep_first, lo) : 0;
+    const int nk = EXT && window > 0 ? min(keep_first, lo) : 0;
     const int total = nk + pos - lo + 1;
     const int ntiles = (total - 1) / KT + 1;
 
-    auto load_tile = [&](int it, int st) {
-        unsigned char* K = Ws + st * stage_bytes;
-        unsigned char* V = K + KT * PK;
-        // lane l < KT finds row l of the tile; the copies then take whole rows with neighbouring lanes
+    // lane l < KT looks up where row l of tile `it` lies in the cache (-1: past the visible keys); the copies then take whole rows with
+    // LPR neighbouring lanes, one 16-byte piece of the key and of the value each
+    constexpr int LPR = DMAX / 8, RPI = 32 / LPR;
+    const int piece = lane % LPR;
+    const bool has_k = piece * 8 < dk, has_v = !shared_kv && piece * 8 < dv;
+    const int k_elem = (shared_kv ? shared_kv_key_offset(G) : 0) + g * dk + piece * 8, v_elem = G * dk + (g / vshare) * dv + piece * 8;
+    auto find_row = [&](int it) -> int {
         const int e = it * KT + lane;
-        const bool ok = lane < KT && e < total;
-        long long row = 0;
-        if (ok) {
-            const int kp = key_position(e, nk, lo), b = kp / block_size;
-            row = (((long long)bt[b] * n_slots + slot) * block_size + (kp - b * block_size)) * row_elems;
-        }
+        if (lane >= KT || e >= total) return -1;
+        const int kp = key_position(e, nk, lo), b = kp / block_size;
+        return (bt[b] * n_slots + slot) * block_size + (kp - b * block_size);  // cache rows are numbered below 2^31
+    };
+    auto load_tile = [&](int row, int st) {
+        const uint32_t K = ws_a + st * stage_bytes, V = K + KT * PK;
         if (shared_kv && lane < KT) {
-            float* ki = reinterpret_cast<float*>(V) + lane;
-            if (ok) cp_async4(smem_u32(ki), cache + row + 2 * g);
-            else *ki = 0.f;
+            if (row >= 0) cp_async4(V + lane * 4, cache + (int64_t)row * row_elems + 2 * g);
+            else *reinterpret_cast<float*>(Ws + st * stage_bytes + KT * PK + lane * 4) = 0.f;
         }
-        const unsigned live = __ballot_sync(0xffffffffu, ok);
-        for (int r0 = 0; r0 < KT; r0 += 32 / lprk) {
-            const int r = r0 + lane / lprk;
-            const long long base = __shfl_sync(0xffffffffu, row, r & 31);
-            const int nb = (live >> (r & 31)) & 1 ? 16 : 0;
-            if (r < KT)
-                for (int ch = lane % lprk; ch < ck; ch += lprk) cp_async16(smem_u32(K + r * PK + ch * 16), cache + base + (nb ? koff + ch * 8 : 0), nb);
+#pragma unroll
+        for (int i = 0; i < KT / RPI; i++) {
+            const int r = i * RPI + lane / LPR;
+            const int src = __shfl_sync(0xffffffffu, row, r);
+            const T* base = cache + (int64_t)max(src, 0) * row_elems;
+            const int nb = src >= 0 ? 16 : 0;
+            if (has_k) cp_async16(K + r * PK + piece * 16, base + k_elem, nb);
+            if (has_v) cp_async16(V + r * PV + piece * 16, base + v_elem, nb);
         }
-        if (!shared_kv)
-            for (int r0 = 0; r0 < KT; r0 += 32 / lprv) {
-                const int r = r0 + lane / lprv;
-                const long long base = __shfl_sync(0xffffffffu, row, r & 31);
-                const int nb = (live >> (r & 31)) & 1 ? 16 : 0;
-                if (r < KT)
-                    for (int ch = lane % lprv; ch < cv; ch += lprv) cp_async16(smem_u32(V + r * PV + ch * 16), cache + base + (nb ? voff + ch * 8 : 0), nb);
-            }
         cp_async_commit();
     };
-    if (warp < ntiles) load_tile(warp, 0);
+    int row_next = warp < ntiles ? find_row(warp) : -1;
+#pragma unroll
+    for (int i = 0; i < WD_STAGES - 1; i++) {
+        const int it = warp + i * WD_WARPS;
+        if (it < ntiles) { load_tile(row_next, i); row_next = it + WD_WARPS < ntiles ? find_row(it + WD_WARPS) : -1; }
+        else cp_async_commit();                                                // an empty group keeps the count
+    }
 
     // ---- queries: rows past the group's heads are zeros; eight threads per row
     {
@@ -711,118 +719,165 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(
         }
     }
     __syncthreads();
-    uint32_t qf[DMAX / 16][4];
+    uint32_t qf[DMAX / 16][NH][2];                                             // Q^T as B fragments: heads 8 n .. 8 n + 7
 #pragma unroll
     for (int kk = 0; kk < DMAX / 16; kk++)
-        if (kk * 16 < dk)
-            ldmatrix_x4(smem_u32(Qs + ((lane & 7) + ((lane >> 3) & 1) * 8) * PQ + (kk * 16 + (lane >> 4) * 8) * 2), qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3]);
+        if (kk * 16 < dk) {
+            uint32_t b0, b1, b2, b3;
+            ldmatrix_x4(smem_u32(Qs + ((lane & 7) + (lane >> 4) * 8) * PQ + (kk * 16 + ((lane >> 3) & 1) * 8) * 2), b0, b1, b2, b3);
+            qf[kk][0][0] = b0; qf[kk][0][1] = b1;
+            if constexpr (NH == 2) { qf[kk][1][0] = b2; qf[kk][1][1] = b3; }
+        }
 
-    const int r_a = lane >> 2, r_b = r_a + 8;
+    // this lane's heads: 8 n + 2 (lane % 4) + e; its keys within a 16-key block: lane / 4 and lane / 4 + 8
     const float cap_in = softcap > 0.f ? scale_log2 * 0.6931471805599453f / softcap : 0.f;
     const float cap_out = softcap * 1.4426950408889634f;
-    const float sl_a = slopes != nullptr && r_a < hq ? slopes[g * hq + r_a] * 1.4426950408889634f : 0.f;
-    const float sl_b = slopes != nullptr && r_b < hq ? slopes[g * hq + r_b] * 1.4426950408889634f : 0.f;
-    float m_a = sink > 0.f && warp == 0 ? 0.f : -INFINITY, m_b = m_a;
-    float l_a = (lane & 3) == 0 && warp == 0 ? sink : 0.f, l_b = l_a;
-    float o[DMAX / 8][4];
+    float m[NH][2], l[NH][2], sl[NH][2];
 #pragma unroll
-    for (int nt = 0; nt < DMAX / 8; nt++) { o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f; }
+    for (int n = 0; n < NH; n++)
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+            const int hh = n * 8 + 2 * (lane & 3) + e;
+            m[n][e] = sink > 0.f && warp == 0 ? 0.f : -INFINITY;
+            l[n][e] = lane < 4 && warp == 0 ? sink : 0.f;
+            sl[n][e] = slopes != nullptr && hh < hq ? slopes[g * hq + hh] * 1.4426950408889634f : 0.f;
+        }
+    float o[DMAX / 16][NH][4];
+#pragma unroll
+    for (int mt = 0; mt < DMAX / 16; mt++)
+#pragma unroll
+        for (int n = 0; n < NH; n++) { o[mt][n][0] = o[mt][n][1] = o[mt][n][2] = o[mt][n][3] = 0.f; }
 
     int st = 0;
-    for (int it = warp; it < ntiles; it += WD_WARPS, st ^= 1) {
-        if (it + WD_WARPS < ntiles) { load_tile(it + WD_WARPS, st ^ 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
+    for (int it = warp; it < ntiles; it += WD_WARPS) {
+        {
+            const int ahead = it + (WD_STAGES - 1) * WD_WARPS;
+            const int st_ahead = st + WD_STAGES - 1 >= WD_STAGES ? st - 1 : st + WD_STAGES - 1;
+            if (ahead < ntiles) {
+                load_tile(row_next, st_ahead);
+                row_next = ahead + WD_WARPS < ntiles ? find_row(ahead + WD_WARPS) : -1;
+            } else {
+                cp_async_commit();
+            }
+        }
+        cp_async_wait<WD_STAGES - 1>();
         __syncwarp();                                                          // the tile is visible to the whole warp
-        const unsigned char* Kt = Ws + st * stage_bytes;
-        const unsigned char* Vt = shared_kv ? Kt : Kt + KT * PK;
+        const uint32_t Kt = ws_a + st * stage_bytes, Vt = shared_kv ? Kt : Kt + KT * PK;
         const int PVt = shared_kv ? PK : PV;
-        float sc[KT / 8][4];
+        float sc[KT / 16][NH][4];
 #pragma unroll
-        for (int nt = 0; nt < KT / 8; nt++) { sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f; }
+        for (int b = 0; b < KT / 16; b++)
+#pragma unroll
+            for (int n = 0; n < NH; n++) { sc[b][n][0] = sc[b][n][1] = sc[b][n][2] = sc[b][n][3] = 0.f; }
+        const uint32_t k_addr = Kt + ((lane & 7) + ((lane >> 3) & 1) * 8) * PK + (lane >> 4) * 16;
 #pragma unroll
         for (int kk = 0; kk < DMAX / 16; kk++) {
             if (kk * 16 < dk) {
 #pragma unroll
-                for (int np = 0; np < KT / 16; np++) {
-                    uint32_t b0, b1, b2, b3;
-                    ldmatrix_x4(smem_u32(Kt + (np * 16 + (lane >> 4) * 8 + (lane & 7)) * PK + (kk * 16 + ((lane >> 3) & 1) * 8) * 2), b0, b1, b2, b3);
-                    mma_16816<T>(sc[2 * np], qf[kk], b0, b1);
-                    mma_16816<T>(sc[2 * np + 1], qf[kk], b2, b3);
+                for (int b = 0; b < KT / 16; b++) {
+                    uint32_t a[4];
+                    ldmatrix_x4(k_addr + b * 16 * PK + kk * 32, a[0], a[1], a[2], a[3]);
+#pragma unroll
+                    for (int n = 0; n < NH; n++) mma_16816<T>(sc[b][n], a, qf[kk][n][0], qf[kk][n][1]);
                 }
             }
         }
-        const float* ki = reinterpret_cast<const float*>(Kt + KT * PK) + (lane & 3) * 2;
-        float mx_a = -INFINITY, mx_b = -INFINITY;
+        float mx[NH][2];
 #pragma unroll
-        for (int nt = 0; nt < KT / 8; nt++) {
-            if (shared_kv) {
-                const float2 f = *reinterpret_cast<const float2*>(ki + nt * 8);
-                sc[nt][0] *= f.x; sc[nt][1] *= f.y; sc[nt][2] *= f.x; sc[nt][3] *= f.y;
+        for (int n = 0; n < NH; n++) { mx[n][0] = mx[n][1] = -INFINITY; }
+        const float* ki = reinterpret_cast<const float*>(Ws + st * stage_bytes + KT * PK) + (lane >> 2);
+#pragma unroll
+        for (int b = 0; b < KT / 16; b++) {
+#pragma unroll
+            for (int half = 0; half < 2; half++) {
+                const int v = it * KT + b * 16 + half * 8 + (lane >> 2);       // every entry of the list below `total` is visible
+                const float kinv = shared_kv ? ki[b * 16 + half * 8] : 1.f;
+                const float dist = EXT ? (float)(pos - key_position(v, nk, lo)) : 0.f;
+#pragma unroll
+                for (int n = 0; n < NH; n++)
+#pragma unroll
+                    for (int e = 0; e < 2; e++) {
+                        float x = sc[b][n][2 * half + e];
+                        if (shared_kv) x *= kinv;
+                        x = softcap > 0.f ? cap_out * tanhf(x * cap_in) : x * scale_log2;
+                        if (EXT) x -= sl[n][e] * dist;
+                        x = v < total ? x : -INFINITY;
+                        sc[b][n][2 * half + e] = x;
+                        mx[n][e] = fmaxf(mx[n][e], x);
+                    }
             }
+        }
+        float al[NH][2];
+#pragma unroll
+        for (int n = 0; n < NH; n++)
 #pragma unroll
             for (int e = 0; e < 2; e++) {
-                const int v = it * KT + nt * 8 + (lane & 3) * 2 + e;           // every entry of the list below `total` is visible
-                float sa = softcap > 0.f ? cap_out * tanhf(sc[nt][e] * cap_in) : sc[nt][e] * scale_log2;
-                float sb = softcap > 0.f ? cap_out * tanhf(sc[nt][2 + e] * cap_in) : sc[nt][2 + e] * scale_log2;
-                if (EXT) {
-                    const float dist = (float)(pos - key_position(v, nk, lo));
-                    sa -= sl_a * dist;
-                    sb -= sl_b * dist;
-                }
-                sc[nt][e] = v < total ? sa : -INFINITY;
-                sc[nt][2 + e] = v < total ? sb : -INFINITY;
-                mx_a = fmaxf(mx_a, sc[nt][e]);
-                mx_b = fmaxf(mx_b, sc[nt][2 + e]);
+                float x = mx[n][e];
+                x = fmaxf(x, __shfl_xor_sync(0xffffffffu, x, 4));
+                x = fmaxf(x, __shfl_xor_sync(0xffffffffu, x, 8));
+                x = fmaxf(x, __shfl_xor_sync(0xffffffffu, x, 16));
+                x = fmaxf(x, m[n][e]);                                         // finite: a tile has at least one visible key
+                al[n][e] = exp2f(m[n][e] - x);
+                m[n][e] = x;
+                l[n][e] *= al[n][e];
             }
-        }
-        mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 1)); mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 2));
-        mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 1)); mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 2));
-        const float mn_a = fmaxf(m_a, mx_a), mn_b = fmaxf(m_b, mx_b);          // finite: a tile has at least one visible key
-        const float al_a = exp2f(m_a - mn_a), al_b = exp2f(m_b - mn_b);
-        m_a = mn_a; m_b = mn_b;
-        l_a *= al_a; l_b *= al_b;
 #pragma unroll
-        for (int nt = 0; nt < DMAX / 8; nt++) { o[nt][0] *= al_a; o[nt][1] *= al_a; o[nt][2] *= al_b; o[nt][3] *= al_b; }
-        uint32_t pa[KT / 16][4];
+        for (int mt = 0; mt < DMAX / 16; mt++)
 #pragma unroll
-        for (int nt = 0; nt < KT / 8; nt++) {
-            const float p0 = exp2f(sc[nt][0] - mn_a), p1 = exp2f(sc[nt][1] - mn_a);
-            const float p2 = exp2f(sc[nt][2] - mn_b), p3 = exp2f(sc[nt][3] - mn_b);
-            l_a += p0 + p1; l_b += p2 + p3;
-            pa[nt >> 1][(nt & 1) * 2] = pack2<T>(p0, p1);
-            pa[nt >> 1][(nt & 1) * 2 + 1] = pack2<T>(p2, p3);
-        }
+            for (int n = 0; n < NH; n++) {
+                o[mt][n][0] *= al[n][0]; o[mt][n][1] *= al[n][1]; o[mt][n][2] *= al[n][0]; o[mt][n][3] *= al[n][1];
+            }
+        const uint32_t v_addr = Vt + ((lane & 7) + (lane >> 4) * 8) * PVt + ((lane >> 3) & 1) * 16;
 #pragma unroll
-        for (int kk = 0; kk < KT / 16; kk++) {
+        for (int b = 0; b < KT / 16; b++) {                                    // 16 keys per step
+            uint32_t pb[NH][2];
 #pragma unroll
-            for (int np = 0; np < DMAX / 16; np++) {
-                if (np * 16 < dv) {
-                    uint32_t b0, b1, b2, b3;
-                    ldmatrix_x4_trans(smem_u32(Vt + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PVt + (np * 16 + (lane >> 4) * 8) * 2), b0, b1, b2, b3);
-                    mma_16816<T>(o[2 * np], pa[kk], b0, b1);
-                    mma_16816<T>(o[2 * np + 1], pa[kk], b2, b3);
+            for (int n = 0; n < NH; n++)
+#pragma unroll
+                for (int half = 0; half < 2; half++) {
+                    const float p0 = exp2f(sc[b][n][2 * half] - m[n][0]), p1 = exp2f(sc[b][n][2 * half + 1] - m[n][1]);
+                    l[n][0] += p0; l[n][1] += p1;
+                    pb[n][half] = movmatrix_trans(pack2<T>(p0, p1));
+                }
+#pragma unroll
+            for (int mt = 0; mt < DMAX / 16; mt++) {
+                if (mt * 16 < dv) {
+                    uint32_t a[4];
+                    ldmatrix_x4_trans(v_addr + b * 16 * PVt + mt * 32, a[0], a[1], a[2], a[3]);
+#pragma unroll
+                    for (int n = 0; n < NH; n++) mma_16816<T>(o[mt][n], a, pb[n][0], pb[n][1]);
                 }
             }
         }
         __syncwarp();                                                          // the stage may be overwritten
+        st = st + 1 == WD_STAGES ? 0 : st + 1;
     }
 
     // ---- merge the warps, (turn back,) gate, store
-    l_a += __shfl_xor_sync(0xffffffffu, l_a, 1); l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
-    l_b += __shfl_xor_sync(0xffffffffu, l_b, 1); l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
+    cp_async_wait<0>();
     __syncthreads();                                                           // every warp is done with its tiles
     float* Om = reinterpret_cast<float*>(smem_raw);                            // [WD_WARPS][hq][dv]
     float* Ms = Om + WD_WARPS * hq * dv;                                       // [WD_WARPS][16] maximum, then [WD_WARPS][16] sum
 #pragma unroll
-    for (int e = 0; e < 2; e++) {
-        const int r = e ? r_b : r_a;
-        if (r >= hq) continue;
-        if ((lane & 3) == 0) { Ms[warp * 16 + r] = e ? m_b : m_a; Ms[(WD_WARPS + warp) * 16 + r] = e ? l_b : l_a; }
+    for (int n = 0; n < NH; n++)
 #pragma unroll
-        for (int nt = 0; nt < DMAX / 8; nt++) {
-            const int d = nt * 8 + (lane & 3) * 2;
-            if (d < dv) *reinterpret_cast<float2*>(Om + (warp * hq + r) * dv + d) = make_float2(o[nt][2 * e], o[nt][2 * e + 1]);
+        for (int e = 0; e < 2; e++) {
+            float x = l[n][e];
+            x += __shfl_xor_sync(0xffffffffu, x, 4);
+            x += __shfl_xor_sync(0xffffffffu, x, 8);
+            x += __shfl_xor_sync(0xffffffffu, x, 16);
+            const int hh = n * 8 + 2 * (lane & 3) + e;
+            if (hh >= hq) continue;
+            if (lane < 4) { Ms[warp * 16 + hh] = m[n][e]; Ms[(WD_WARPS + warp) * 16 + hh] = x; }
+#pragma unroll
+            for (int mt = 0; mt < DMAX / 16; mt++) {
+                const int d = mt * 16 + (lane >> 2);
+                if (mt * 16 < dv) {
+                    Om[(warp * hq + hh) * dv + d] = o[mt][n][e];
+                    Om[(warp * hq + hh) * dv + d + 8] = o[mt][n][2 + e];
+                }
+            }
         }
-    }
     __syncthreads();
     const int n_out = hq * dv;
     for (int i = tid; i < n_out; i += WD_WARPS * 32) {                         // slot 0 <- the normalised output
@@ -916,9 +971,10 @@ static int launch_window_attn_mma(const void* q, int64_t q_stride_t, const void*
     auto kern_decode = window_attn_mma_kernel<T, DMAX, 64, EXT>;
     // single decoded tokens of up to 16 heads per group: keys split over the warps of a CTA; small tiles where a row is long
     constexpr int KT = DMAX == 64 || EXT ? 32 : 16;
-    auto kern_split = window_attn_decode_kernel<T, DMAX, KT, EXT>;
+    auto kern_split = hq <= 8 ? window_attn_decode_kernel<T, DMAX, KT, 1, EXT> : window_attn_decode_kernel<T, DMAX, KT, 2, EXT>;
     if (first_use_on_this_device(attr_mask)) {
-        cudaFuncSetAttribute(kern_split, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+        cudaFuncSetAttribute(window_attn_decode_kernel<T, DMAX, KT, 1, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+        cudaFuncSetAttribute(window_attn_decode_kernel<T, DMAX, KT, 2, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
         cudaFuncSetAttribute(kern_prompt, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);
         cudaFuncSetAttribute(kern_decode, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);
     }
@@ -930,7 +986,7 @@ static int launch_window_attn_mma(const void* q, int64_t q_stride_t, const void*
         const int64_t first = parts[k][0], count = parts[k][1];
         if (count <= 0) continue;
         if (k == 1 && hq <= 16) {
-            size_t smem = 16 * (size_t)(dk * 2 + 16) + WD_WARPS * 2 * (size_t)KT * ((dk * 2 + 16) + (shared_kv ? sizeof(float) : dv * 2 + 16));
+            size_t smem = 16 * (size_t)(dk * 2 + 16) + WD_WARPS * WD_STAGES * (size_t)KT * ((dk * 2 + 16) + (shared_kv ? sizeof(float) : dv * 2 + 16));
             const size_t merge = ((size_t)WD_WARPS * hq * dv + 2 * WD_WARPS * 16) * sizeof(float);
             if (smem < merge) smem = merge;
             kern_split<<<dim3((unsigned)count, (unsigned)G), WD_WARPS * 32, smem, stream>>>(

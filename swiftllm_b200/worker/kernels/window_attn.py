@@ -87,6 +87,7 @@ def window_attention(q: torch.Tensor, gate, cache: torch.Tensor, slot: int, bloc
     assert gate is None or (gate.shape == (T, heads if opt.gate_per_head else heads * dv) and gate.stride(1) == 1 and gate.dtype == q.dtype)
     row = shared_row_width(kv_heads, dk) if opt.shared_kv else kv_heads * dk + kv_heads // opt.vshare * dv
     assert cache.shape[3] == row and cache.dtype == q.dtype and (not opt.shared_kv or dk == dv)
+    assert cache.shape[0] * cache.shape[1] * cache.shape[2] < 1 << 31       # rows are numbered in 32 bits
     assert opt.slopes is None or (opt.slopes.dtype == torch.float32 and opt.slopes.shape == (heads,))
     assert out.dtype == (torch.float32 if opt.out_f32 else q.dtype)
     assert opt.q_norm is None or (opt.q_norm.dtype == torch.float32 and opt.q_norm.shape == (dk,))
