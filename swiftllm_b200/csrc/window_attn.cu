@@ -604,12 +604,11 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
 }
 
 // ------------------------------------------------------------------ attention of single decoded tokens (tensor cores, 16-bit storage)
-// One CTA = one token and key/value group of at most 8 NH query heads.  The token's visible keys are split over the CTA's four WARPS:
-// warp w walks the tiles w, w + 4, .. of KT keys through a cp.async ring of its own (no CTA barrier inside the loop) with its own
-// running (maximum, sum, output); the four results are merged through shared memory at the end.  The products are taken transposed, so
+// One CTA = one token and key/value group of at most 8 NH query heads.  The token's visible keys are split over the CTA's
+// WARPS (4 or 8): warp w walks the tiles w, w + WD_WARPS, .. of KT keys through a cp.async ring of its own (no CTA barrier inside the loop) with its own
+// running (maximum, sum, output); the results are merged through shared memory at the end.  The products are taken transposed, so
 // that the few heads are the narrow side of the MMA tiles: S^T [keys, heads] = K Q^T with Q^T in registers for the whole walk, then
 // O^T [dv, heads] += V^T P^T, where P^T is S^T's fragment turned by movmatrix.  Same options as the kernel above.
-constexpr int WD_WARPS = 4;
 constexpr int WD_STAGES = 3;
 
 // the 8 x 8 matrix of 16-bit entries held by the warp, transposed
@@ -619,7 +618,7 @@ __device__ __forceinline__ uint32_t movmatrix_trans(uint32_t x) {
     return y;
 }
 
-template <typename T, int DMAX, int KT, int NH, bool EXT>
+template <typename T, int DMAX, int KT, int NH, int WD_WARPS, bool EXT>
 __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(
     const T* __restrict__ q, int64_t q_stride_t, const float* __restrict__ cosb, const float* __restrict__ sinb,
     const T* __restrict__ gate, int64_t gate_stride_t, const T* __restrict__ cache, int n_slots, int slot, int block_size,
@@ -687,9 +686,10 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(
         else cp_async_commit();                                                // an empty group keeps the count
     }
 
-    // ---- queries: rows past the group's heads are zeros; eight threads per row
+    // ---- queries: rows past the group's heads are zeros
     {
-        const int r = tid >> 3, part = tid & 7;
+        constexpr int TPR = WD_WARPS * 2;                                      // threads per row (16 rows)
+        const int r = tid / TPR, part = tid % TPR;
         const bool live = r < hq;
         const int half = rot_dims >> 1;
         const T* qr = q + t * q_stride_t + (int64_t)(g * hq + (live ? r : 0)) * dk;
@@ -698,18 +698,20 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(
         float pinv = 1.f;
         if (qnorm_w != nullptr) {
             float s0 = 0.f;
-            for (int i = part; i < dk; i += 8) { const float a = ldf(qr + i); s0 += a * a; }
+            for (int i = part; i < dk; i += TPR) { const float a = ldf(qr + i); s0 += a * a; }
             s0 += __shfl_xor_sync(0xffffffffu, s0, 1); s0 += __shfl_xor_sync(0xffffffffu, s0, 2); s0 += __shfl_xor_sync(0xffffffffu, s0, 4);
+            if constexpr (TPR == 16) s0 += __shfl_xor_sync(0xffffffffu, s0, 8);
             pinv = 1.f / sqrtf(s0 / (float)dk + prenorm_eps);
         }
         float inv = 1.f;
         if (qk_norm_eps >= 0.f) {
             float ss = 0.f;
-            for (int i = part; i < dk; i += 8) { const float a = rot_entry(qr, i, rot_dims, halves, cs, sn, pinv, qnorm_w); ss += a * a; }
+            for (int i = part; i < dk; i += TPR) { const float a = rot_entry(qr, i, rot_dims, halves, cs, sn, pinv, qnorm_w); ss += a * a; }
             ss += __shfl_xor_sync(0xffffffffu, ss, 1); ss += __shfl_xor_sync(0xffffffffu, ss, 2); ss += __shfl_xor_sync(0xffffffffu, ss, 4);
+            if constexpr (TPR == 16) ss += __shfl_xor_sync(0xffffffffu, ss, 8);
             inv = 1.f / sqrtf(ss / (float)dk + qk_norm_eps);
         }
-        for (int i = part; i < (dk >> 1); i += 8) {
+        for (int i = part; i < (dk >> 1); i += TPR) {
             float a = 0.f, b = 0.f;
             if (live) {
                 a = rot_entry(qr, 2 * i, rot_dims, halves, cs, sn, pinv, qnorm_w) * inv;
@@ -970,11 +972,12 @@ static int launch_window_attn_mma(const void* q, int64_t q_stride_t, const void*
     auto kern_prompt = window_attn_mma_kernel<T, DMAX, 32, EXT>;
     auto kern_decode = window_attn_mma_kernel<T, DMAX, 64, EXT>;
     // single decoded tokens of up to 16 heads per group: keys split over the warps of a CTA; small tiles where a row is long
-    constexpr int KT = DMAX == 64 || EXT ? 32 : 16;
-    auto kern_split = hq <= 8 ? window_attn_decode_kernel<T, DMAX, KT, 1, EXT> : window_attn_decode_kernel<T, DMAX, KT, 2, EXT>;
+    // (eight warps where a key row is also the value row and a stage is half as large)
+    constexpr int KT = DMAX == 64 ? 32 : 16, WD_WARPS = EXT ? 8 : 4;
+    auto kern_split = hq <= 8 ? window_attn_decode_kernel<T, DMAX, KT, 1, WD_WARPS, EXT> : window_attn_decode_kernel<T, DMAX, KT, 2, WD_WARPS, EXT>;
     if (first_use_on_this_device(attr_mask)) {
-        cudaFuncSetAttribute(window_attn_decode_kernel<T, DMAX, KT, 1, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
-        cudaFuncSetAttribute(window_attn_decode_kernel<T, DMAX, KT, 2, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+        cudaFuncSetAttribute(window_attn_decode_kernel<T, DMAX, KT, 1, WD_WARPS, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+        cudaFuncSetAttribute(window_attn_decode_kernel<T, DMAX, KT, 2, WD_WARPS, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
         cudaFuncSetAttribute(kern_prompt, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);
         cudaFuncSetAttribute(kern_decode, cudaFuncAttributeMaxDynamicSharedMemorySize, 120 * 1024);
     }
