@@ -267,13 +267,23 @@ __global__ void __launch_bounds__(256) gla_chunk_scan_kernel(const float* __rest
     float S = tok_pos[seg0] > 0 ? state[((int64_t)seq_ids[b] * H + h) * size + i] : 0.f;
     float* p = chunk_states + (((int64_t)b * chunks) * H + h) * size + i;
     const float* a = chunk_decays + (((int64_t)b * chunks) * H + h) * dk + d;
-    for (int c = 0; c < live; c++) {
-        const bool more = c + 1 < live;                                 // the last chunk left no contribution
-        const float add = more ? *p : 0.f, f = more ? *a : 0.f;
-        *p = S;
-        S = f * S + add;
-        p += H * size;
-        a += (int64_t)H * dk;
+    const int64_t step = H * size;
+    constexpr int AHEAD = 8;                                            // contributions in flight
+    for (int c0 = 0; c0 < live; c0 += AHEAD) {
+        float add[AHEAD], f[AHEAD];
+#pragma unroll
+        for (int j = 0; j < AHEAD; j++) {
+            const bool more = c0 + j + 1 < live;                        // the last chunk left no contribution
+            add[j] = more ? p[j * step] : 0.f;
+            f[j] = more ? a[(int64_t)j * H * dk] : 0.f;
+        }
+#pragma unroll
+        for (int j = 0; j < AHEAD; j++) {
+            if (c0 + j < live) p[j * step] = S;
+            S = f[j] * S + add[j];
+        }
+        p += AHEAD * step;
+        a += (int64_t)AHEAD * H * dk;
     }
 }
 
