@@ -200,7 +200,7 @@ def _windowed_step(H, G, d, dtype, g, bs=16):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,G,d,window,keep", [(4, 2, 32, 64, 4), (8, 1, 64, 50, 0), (6, 3, 48, 33, 40), (10, 10, 16, 7, 1), (6, 2, 128, 1000, 5),
-                                               (3, 1, 80, 1, 2), (6, 2, 10, 20, 3), (5, 5, 7, 9, 2), (2, 1, 200, 30, 6)])
+                                               (12, 1, 48, 60, 2), (32, 2, 112, 90, 3), (18, 1, 32, 25, 4), (3, 1, 80, 1, 2), (6, 2, 10, 20, 3), (5, 5, 7, 9, 2), (2, 1, 200, 30, 6)])
 def test_window_attention_whose_values_are_its_keys(dtype, H, G, d, window, keep):
     """Both attention kernels on the same step (the CUDA-core one is forced for the second run) and a plain loop: kept first
     positions, distance bias, norm of keys and queries, un-normed keys as values, one gate per head."""
