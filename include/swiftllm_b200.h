@@ -307,7 +307,19 @@ int sllm_window_kv_store(const void* k, int64_t k_row_stride, const void* v, int
  * and cap.  keep_first > 0 (with a window, without chunks): positions 0 .. keep_first - 1 stay visible.  gate_per_head = 1: gate
  * is [T, num_heads].  shared_kv = 1: the values are the un-normed keys (dk = dv, no rotation); a cache row (written by
  * shared_kv_store) is [1 / rms of every key head, fp32, 2 num_kv_heads elements rounded up to 8 | keys as projected, num_kv_heads *
- * dk elements rounded up to 8] and s_j uses key / rms(key); a key norm's weight is folded into qnorm_w by the caller. */
+ * dk elements rounded up to 8] and s_j uses key / rms(key); a key norm's weight is folded into qnorm_w by the caller.
+ * sinks (fp32 [num_heads], or NULL; not with sink = 1): the denominator also contains exp(sinks[h]).  krot > 0 (with shared_kv): rows
+ * and queries as whole_norm_rope_store writes them.
+ * whole_norm_rope_store: q [T, num_heads * dk] and k [T, num_kv_heads * dk] are RMS-normed over their whole rows (weights fp32
+ * q_norm_w [num_heads * dk], k_norm_w [num_kv_heads * dk]) and turned on the first rot_dims entries of every head; the values are the
+ * un-normed keys.  The cache row is [1 / rms of k, fp32, num_kv_heads times, 2 num_kv_heads elements rounded up to 8 | per key head: dk
+ * entries as projected, then rot_dims turned entries of k * k_norm_w; rounded up to 8]; q_out [T, num_heads, dk] = per head [entries
+ * rot_dims .. dk - 1 of the normed query times k_norm_w | the turned entries], for window_attention with krot = rot_dims. */
+int sllm_whole_norm_rope_store(const void* q, int64_t q_row_stride, const void* k, int64_t k_row_stride, const void* q_norm_w,
+                               const void* k_norm_w, float eps, const void* cosb, const void* sinb, const void* tok_seq,
+                               const void* tok_pos, const void* block_table, int max_blocks_per_seq, void* cache, int n_slots, int slot,
+                               int block_size, void* q_out, int64_t num_tokens, int num_heads, int num_kv_heads, int dk, int rot_dims,
+                               int pair_halves, sllm_dtype_t dtype, sllm_stream_t stream);
 int sllm_shared_kv_store(const void* k, int64_t k_row_stride, const void* tok_seq, const void* tok_pos, const void* block_table,
                          int max_blocks_per_seq, void* cache, int n_slots, int slot, int block_size, int64_t num_tokens,
                          int num_kv_heads, int dk, float eps, sllm_dtype_t dtype, sllm_stream_t stream);
@@ -319,7 +331,7 @@ int sllm_window_attention(const void* q, int64_t q_stride_t, const void* cosb, c
                           int dk, int dv, int rot_dims, int window, float scale, int sink, int pair_halves, float qk_norm_eps,
                           float softcap, const void* vcos, const void* vsin, float out_scale, const void* qnorm_w,
                           float prenorm_eps, int chunk, int vshare, int out_f32, const void* slopes, int keep_first,
-                          int gate_per_head, int shared_kv, sllm_dtype_t dtype, sllm_stream_t stream);
+                          int gate_per_head, int shared_kv, int krot, const void* sinks, sllm_dtype_t dtype, sllm_stream_t stream);
 /* diff_combine: a fp32 [T, num_kv_heads, 2, num_heads / num_kv_heads, dv] - the outputs of two score maps per head over the same
  * values (window_attention with vshare = 2, 2 * num_heads queries ordered [key/value head][map][head of the group], out_f32).
  * out[t, h] = o / sqrt(mean(o^2) + eps) * factor * sigmoid(gate[t, h]) with o = a[map 0] - lambda * a[map 1]; gate logits
@@ -332,7 +344,7 @@ int sllm_diff_combine(const void* a, const void* gate, int64_t gate_stride_t, vo
  * embed_pair_hash: x[t] (fp32) = embed[tokens[t]] * scale + pairs[row], row = (previous * mul_prev + token * mul_cur) mod buckets with
  * `previous` the token one position earlier (the row above, or last_token[tok_seq[t]] (int32 per sequence row) when the step
  * starts there); a token at position 0 takes row `buckets`.  pairs may be NULL (no pair table).  x_copy (fp32, may be NULL)
- * gets the same values; h gets their rounding to dtype.  store_last_tokens then records every segment's last token. */
+ * gets the same values; h (may be NULL) gets their rounding to dtype.  store_last_tokens then records every segment's last token. */
 int sllm_embed_pair_hash(const void* tokens, const void* tok_seq, const void* tok_pos, const void* last_token, const void* embed,
                          const void* pairs, int buckets, int64_t mul_prev, int64_t mul_cur, float scale, void* x, void* x_copy,
                          void* h, int64_t num_tokens, int width, sllm_dtype_t dtype, sllm_stream_t stream);
@@ -351,10 +363,11 @@ int sllm_sigmoid_gate_inplace(void* x, const void* gate, int64_t gate_stride, in
                               sllm_stream_t stream);
 int sllm_tanh_cap_inplace(void* x, int64_t n, float cap, sllm_dtype_t dtype, sllm_stream_t stream);
 /* moe_route_sigmoid: logits fp32 [T, experts] -> weights fp32 [T, experts]: s = sigmoid(logits); the `top` experts with the
- * largest s + bias (fp32 [experts] or NULL) get weight s, the others 0.  moe_silu_glu_scale: u [T, experts * 2 * ff] (per expert
+ * largest s + bias (fp32 [experts] or NULL) get weight s, the others 0; with keep < groups only experts of the `keep` best of `groups`
+ * equal groups of neighbours can be chosen (a group's score: the sum of its two largest s + bias).  moe_silu_glu_scale: u [T, experts * 2 * ff] (per expert
  * [gate | up]) -> y [T, experts * ff] = silu(gate) * up * weights[t, expert]. */
-int sllm_moe_route_sigmoid(const void* logits, const void* bias, void* weights, int64_t num_tokens, int experts, int top,
-                           sllm_stream_t stream);
+int sllm_moe_route_sigmoid(const void* logits, const void* bias, void* weights, int64_t num_tokens, int experts, int top, int groups,
+                           int keep, sllm_stream_t stream);
 int sllm_moe_silu_glu_scale(const void* u, const void* weights, void* y, int64_t num_tokens, int experts, int ff,
                             sllm_dtype_t dtype, sllm_stream_t stream);
 
@@ -395,6 +408,39 @@ int sllm_gla(const void* q, int64_t q_stride, const void* k, int64_t k_stride, c
              int64_t gate_stride, void* state, const void* seg_starts, const void* seq_ids, const void* tok_pos, void* workspace,
              int64_t workspace_floats, void* out, int64_t out_stride, int64_t num_tokens, int64_t num_prefill_tokens, int num_segs,
              int num_prefill_segs, int64_t max_prefill_len, int num_heads, int dk, int dv, sllm_dtype_t dtype, sllm_stream_t stream);
+
+/* ---- Matrix state per head with ONE decay per head and token (new, head_decay.cuh).  Segments, state rows and workspace as above: a step's
+ * first num_prefill_segs segments (num_prefill_tokens rows) are prompt portions, every other segment is one decoded token; workspace:
+ * num_prefill_tokens * num_heads * dv floats (matrix_memory: + num_prefill_segs * num_heads * (dk + 1)).  q, k, v, gate in dtype; gate
+ * logits fp32 [T, num_heads] (row strides in elements); state fp32 [rows, num_heads, dk, dv], in place; dk <= 512, dv <= 4096.
+ * delta_rule: q, k [T, num_kv_heads * dk] are divided by sqrt(sum of squares + 1e-6) per head, q also times q_scale; g = exp(-rate
+ * softplus(decay_logits + decay_bias)), beta = sigmoid(beta_logits); S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q;
+ * out = o / sqrt(mean(o^2) + eps) * norm_w (fp32 [dv]) * silu(gate).
+ * matrix_memory: i = cap tanh((input_logits + input_bias) / cap), f = log sigmoid(cap tanh((forget_logits + forget_bias) / cap)), M =
+ * max(f + m, i); S <- e^(f + m - M) S + e^(i - M) k v^T, n likewise with k, m <- M (norm_state fp32 [rows, num_heads, dk], max_state
+ * fp32 [rows, num_heads]; zero at position 0); o = S^T q / (max(|n . q|, e^-m) + 1e-6) with q times q_scale; out = o / sqrt(mean(o^2) +
+ * eps) * norm_w (fp32 [num_heads * dv]) * sigmoid(gate). */
+int sllm_delta_rule(const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t v_stride,
+                    const void* decay_logits, int64_t decay_stride, const void* beta_logits, int64_t beta_stride, const void* decay_bias,
+                    const void* rate, float q_scale, const void* norm_w, float eps, const void* gate, int64_t gate_stride, void* state,
+                    const void* seg_starts, const void* seq_ids, const void* tok_pos, void* workspace, int64_t workspace_floats,
+                    void* out, int64_t out_stride, int64_t num_tokens, int64_t num_prefill_tokens, int num_segs, int num_prefill_segs,
+                    int num_heads, int num_kv_heads, int dk, int dv, sllm_dtype_t dtype, sllm_stream_t stream);
+int sllm_matrix_memory(const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t v_stride,
+                       const void* forget_logits, int64_t forget_stride, const void* input_logits, int64_t input_stride,
+                       const void* forget_bias, const void* input_bias, float gate_cap, float q_scale, const void* norm_w, float eps,
+                       const void* gate, int64_t gate_stride, void* state, void* norm_state, void* max_state, const void* seg_starts,
+                       const void* seq_ids, const void* tok_pos, void* workspace, int64_t workspace_floats, void* out,
+                       int64_t out_stride, int64_t num_tokens, int64_t num_prefill_tokens, int num_segs, int num_prefill_segs,
+                       int num_heads, int dk, int dv, sllm_dtype_t dtype, sllm_stream_t stream);
+
+/* ---- Several residual streams per token (new, hyper_streams.cu).  Row i is token rows[i] (int32; NULL: i).  x_in fp32 [T, streams, width]
+ * (one_stream = 1: [T, width], every stream equal to it); with y (dtype [T, width]; NULL: unchanged) x_t <- sum_s mix[s, t] x_s + share[t] y
+ * (mix fp32 [from, to], share fp32 [streams]), written to x_out (may be x_in unless one_stream; NULL: not written); with h (dtype, one row
+ * per i; NULL: not wanted) h = rms(sum_s in[s] x_s) * norm_w (fp32 [streams], [width]).  streams <= 16. */
+int sllm_stream_mix_norm(const void* x_in, int one_stream, int streams, const void* y, const void* mix, const void* share,
+                         const void* in, const void* norm_w, float eps, void* x_out, void* h, const void* rows, int64_t num_rows,
+                         int width, sllm_dtype_t dtype, sllm_stream_t stream);
 
 /* ---- Sandwich blocks: x <- x + mult * norm_b(sublayer(norm_a(x))) with RMS norms over `groups` equal consecutive parts of a row
  * (new, sandwich_ops.cu).  group_norm_add_norm: with y (dtype [T, width]) x (fp32, in place) += mult * y / rms_g(y) * wb; with

@@ -10,15 +10,17 @@ drive this LlamaModel.
 """
 from swiftllm_b200.engine_config import EngineConfig
 from swiftllm_b200.model_config import (BupozenModelConfig, BuzaraxModelConfig, LlamaModelConfig, NaforaxModelConfig,
-                                        RivudraModelConfig, ZuzezenModelConfig)
+                                        RivudraModelConfig, VoreraxModelConfig, ZuzezenModelConfig)
 from swiftllm_b200.registry import create_model, load_model_config
 from swiftllm_b200.worker.bupozen_model import BupozenModel
 from swiftllm_b200.worker.buzarax_model import BuzaraxModel
 from swiftllm_b200.worker.model import LlamaModel
 from swiftllm_b200.worker.naforax_model import NaforaxModel
 from swiftllm_b200.worker.rivudra_model import RivudraModel
+from swiftllm_b200.worker.vorerax_model import VoreraxModel
 from swiftllm_b200.worker.zuzezen_model import ZuzezenModel
 
 __all__ = ["EngineConfig", "LlamaModelConfig", "LlamaModel", "BupozenModelConfig", "BupozenModel", "RivudraModelConfig", "RivudraModel",
            "BuzaraxModelConfig", "BuzaraxModel", "NaforaxModelConfig", "NaforaxModel", "ZuzezenModelConfig", "ZuzezenModel",
+           "VoreraxModelConfig", "VoreraxModel",
            "create_model", "load_model_config"]

@@ -59,7 +59,8 @@ SIGNATURES = {
                                   _I, _I, _P]),
     "sllm_window_attention_set_simt": (_I, [_I]),
     "sllm_window_attention": (_I, [_P, _L, _P, _P, _P, _L, _P, _I, _I, _I, _P, _I, _P, _P, _P, _L, _L, _L, _I, _I, _I, _I, _I, _I,
-                                   _F, _I, _I, _F, _F, _P, _P, _F, _P, _F, _I, _I, _I, _P, _I, _I, _I, _I, _P]),
+                                   _F, _I, _I, _F, _F, _P, _P, _F, _P, _F, _I, _I, _I, _P, _I, _I, _I, _I, _P, _I, _P]),
+    "sllm_whole_norm_rope_store": (_I, [_P, _L, _P, _L, _P, _P, _F, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _P, _L, _I, _I, _I, _I, _I, _I, _P]),
     "sllm_shared_kv_store": (_I, [_P, _L, _P, _P, _P, _I, _P, _I, _I, _I, _L, _I, _I, _F, _I, _P]),
     "sllm_diff_combine": (_I, [_P, _P, _L, _P, _L, _L, _I, _I, _I, _F, _F, _F, _I, _P]),
     "sllm_group_norm_add_norm": (_I, [_P, _P, _P, _F, _P, _P, _F, _L, _I, _I, _I, _P]),
@@ -78,9 +79,14 @@ SIGNATURES = {
     "sllm_gla_workspace_floats": (_L, [_L, _I, _L, _I, _I, _I]),
     "sllm_gla": (_I, [_P, _L, _P, _L, _P, _L, _P, _L, _P, _F, _F, _P, _F, _P, _L, _P, _P, _P, _P, _P, _L, _P, _L, _L, _L, _I, _I, _L,
                       _I, _I, _I, _I, _P]),
+    "sllm_delta_rule": (_I, [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _F, _P, _F, _P, _L, _P, _P, _P, _P, _P, _L, _P, _L, _L, _L,
+                             _I, _I, _I, _I, _I, _I, _I, _P]),
+    "sllm_matrix_memory": (_I, [_P, _L, _P, _L, _P, _L, _P, _L, _P, _L, _P, _P, _F, _F, _P, _F, _P, _L, _P, _P, _P, _P, _P, _P, _P, _L, _P,
+                                _L, _L, _L, _I, _I, _I, _I, _I, _I, _P]),
+    "sllm_stream_mix_norm": (_I, [_P, _I, _I, _P, _P, _P, _P, _P, _F, _P, _P, _P, _L, _I, _I, _P]),
     "sllm_postnorm_add_mix": (_I, [_P, _P, _P, _I, _F, _P, _I, _P, _P, _L, _I, _I, _P]),
     "sllm_tanh_cap_inplace": (_I, [_P, _L, _F, _I, _P]),
-    "sllm_moe_route_sigmoid": (_I, [_P, _P, _P, _L, _I, _I, _P]),
+    "sllm_moe_route_sigmoid": (_I, [_P, _P, _P, _L, _I, _I, _I, _I, _P]),
     "sllm_moe_silu_glu_scale": (_I, [_P, _P, _P, _L, _I, _I, _I, _P]),
     "sllm_causal_conv": (_I, [_P, _L, _P, _P, _P, _P, _P, _P, _L, _L, _I, _I, _I, _P]),
     "sllm_rglru_scan": (_I, [_P, _P, _I, _P, _L, _P, _P, _L, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P]),

@@ -37,7 +37,7 @@ __global__ void __launch_bounds__(256) embed_pair_hash_kernel(
         if (pr != nullptr) v += ldf(pr + i);
         x[t * width + i] = v;
         if (x_copy != nullptr) x_copy[t * width + i] = v;
-        stf(h + t * width + i, v);
+        if (h != nullptr) stf(h + t * width + i, v);
     }
 }
 
@@ -172,23 +172,44 @@ __global__ void tanh_cap_kernel(T* __restrict__ x, int64_t n, float cap) {
 }
 
 // One warp per token.  s = sigmoid(logits); the `top` experts with the largest s + bias are chosen (equal values: the lower
-// expert index wins); weights[t, e] = s_e at the chosen experts (not renormalised), 0 elsewhere.
-// Dynamic shared memory: warps * 2 * experts floats.
+// expert index wins); weights[t, e] = s_e at the chosen experts (not renormalised), 0 elsewhere.  groups > 1: only experts of the
+// `keep` best of `groups` equal groups of neighbours can be chosen (a group's score: the sum of its two largest s + bias).
+// Dynamic shared memory: warps * (2 * experts + groups) floats.
 __global__ void __launch_bounds__(128) moe_route_sigmoid_kernel(const float* __restrict__ logits, const float* __restrict__ bias,
                                                                 float* __restrict__ weights, int64_t num_tokens, int experts,
-                                                                int top) {
+                                                                int top, int groups, int keep) {
     extern __shared__ float vals[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int64_t t = (int64_t)blockIdx.x * (blockDim.x >> 5) + warp;
     if (t >= num_tokens) return;
-    float* s = vals + warp * 2 * experts;     // scores
+    float* s = vals + warp * (2 * experts + groups);     // scores
     float* c = s + experts;                   // choice scores
+    float* gs = c + experts;                  // group scores
     for (int e = lane; e < experts; e += 32) {
         s[e] = 1.f / (1.f + expf(-logits[t * experts + e]));
         c[e] = s[e] + (bias != nullptr ? bias[e] : 0.f);
         weights[t * experts + e] = 0.f;
     }
     __syncwarp();
+    if (keep < groups) {
+        const int size = experts / groups;
+        for (int g = lane; g < groups; g += 32) {
+            float a = -INFINITY, b = -INFINITY;           // the two largest
+            for (int e = g * size; e < (g + 1) * size; e++) {
+                const float v = c[e];
+                if (v > a) { b = a; a = v; } else if (v > b) b = v;
+            }
+            gs[g] = size > 1 ? a + b : a;
+        }
+        __syncwarp();
+        for (int g = lane; g < groups; g += 32) {         // a group stays when fewer than `keep` groups are before it
+            int before = 0;
+            for (int o = 0; o < groups; o++) before += gs[o] > gs[g] || (gs[o] == gs[g] && o < g);
+            if (before >= keep)
+                for (int e = g * size; e < (g + 1) * size; e++) c[e] = -INFINITY;
+        }
+        __syncwarp();
+    }
     for (int k = 0; k < top; k++) {
         float best = -INFINITY;
         int bi = 0x7fffffff;
@@ -210,20 +231,28 @@ __global__ void __launch_bounds__(128) moe_route_sigmoid_kernel(const float* __r
 
 // u [T, experts * 2 * ff] holds per expert e the rows [gate_e (ff) | up_e (ff)]; y[t, e * ff + f] = silu(gate) * up * w[t, e]:
 // exact zeros for the experts a token does not use, so ONE down projection over the concatenated experts sums the chosen ones.
-template <typename T>
+// V entries a thread (ff % V == 0: one expert's).
+template <typename T, int V>
 __global__ void moe_silu_glu_scale_kernel(const T* __restrict__ u, const float* __restrict__ w, T* __restrict__ y, int64_t n,
                                           int experts, int ff) {
-    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    const int64_t i = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
     if (i >= n) return;
     const int64_t cols = (int64_t)experts * ff;
     const int64_t t = i / cols;
     const int64_t c = i - t * cols;
     const int e = (int)(c / ff), f = (int)(c - (int64_t)e * ff);
     const float wt = w[t * experts + e];
-    if (wt == 0.f) { stf(y + i, 0.f); return; }
     const T* ur = u + t * 2 * cols + (int64_t)e * 2 * ff;
-    const float g = ldf(ur + f), v = ldf(ur + ff + f);
-    stf(y + i, g / (1.f + expf(-g)) * v * wt);
+    if constexpr (V == 4) {
+        if (wt == 0.f) { Quad<T>::store(y + i, make_float4(0.f, 0.f, 0.f, 0.f)); return; }
+        const float4 g = Quad<T>::load(ur + f), v = Quad<T>::load(ur + ff + f);
+        Quad<T>::store(y + i, make_float4(g.x / (1.f + expf(-g.x)) * v.x * wt, g.y / (1.f + expf(-g.y)) * v.y * wt,
+                                          g.z / (1.f + expf(-g.z)) * v.z * wt, g.w / (1.f + expf(-g.w)) * v.w * wt));
+    } else {
+        if (wt == 0.f) { stf(y + i, 0.f); return; }
+        const float g = ldf(ur + f), v = ldf(ur + ff + f);
+        stf(y + i, g / (1.f + expf(-g)) * v * wt);
+    }
 }
 
 }  // namespace sllm
@@ -237,7 +266,7 @@ int sllm_embed_pair_hash(const void* tokens, const void* tok_seq, const void* to
                          int64_t num_tokens, int width, sllm_dtype_t dtype, sllm_stream_t stream) {
     SLLM_REQUIRE(num_tokens >= 0 && width > 0 && (pairs == nullptr || buckets > 0), "embed_pair_hash: bad shape");
     if (num_tokens == 0) return 0;
-    SLLM_REQUIRE(tokens && tok_seq && tok_pos && embed && x && h && (pairs == nullptr || last_token), "embed_pair_hash: null pointer");
+    SLLM_REQUIRE(tokens && tok_seq && tok_pos && embed && x && (pairs == nullptr || last_token), "embed_pair_hash: null pointer");
     SLLM_DISPATCH_DTYPE_F32(dtype, (embed_pair_hash_kernel<T><<<(unsigned)num_tokens, 256, 0, (cudaStream_t)stream>>>(
         (const int*)tokens, (const int*)tok_seq, (const int*)tok_pos, (const int*)last_token, (const T*)embed, (const T*)pairs,
         buckets, mul_prev, mul_cur, scale, (float*)x, (float*)x_copy, (T*)h, width)));
@@ -314,14 +343,16 @@ int sllm_tanh_cap_inplace(void* x, int64_t n, float cap, sllm_dtype_t dtype, sll
     return check_launch("tanh_cap_inplace");
 }
 
-int sllm_moe_route_sigmoid(const void* logits, const void* bias, void* weights, int64_t num_tokens, int experts, int top,
-                           sllm_stream_t stream) {
+int sllm_moe_route_sigmoid(const void* logits, const void* bias, void* weights, int64_t num_tokens, int experts, int top, int groups,
+                           int keep, sllm_stream_t stream) {
     SLLM_REQUIRE(num_tokens >= 0 && experts > 0 && top > 0 && top <= experts && experts <= 2048,
                  "moe_route_sigmoid: need 0 < top <= experts <= 2048 (got top %d, experts %d)", top, experts);
+    SLLM_REQUIRE(groups >= 1 && experts % groups == 0 && keep >= 1 && keep <= groups && top <= keep * (experts / groups),
+                 "moe_route_sigmoid: %d experts from %d of %d groups of %d", top, keep, groups, experts / (groups > 0 ? groups : 1));
     if (num_tokens == 0) return 0;
     SLLM_REQUIRE(logits && weights, "moe_route_sigmoid: null pointer");
-    moe_route_sigmoid_kernel<<<(unsigned)cdiv(num_tokens, 4), 128, 4 * 2 * experts * sizeof(float), (cudaStream_t)stream>>>(
-        (const float*)logits, (const float*)bias, (float*)weights, num_tokens, experts, top);
+    moe_route_sigmoid_kernel<<<(unsigned)cdiv(num_tokens, 4), 128, 4 * (2 * experts + groups) * sizeof(float), (cudaStream_t)stream>>>(
+        (const float*)logits, (const float*)bias, (float*)weights, num_tokens, experts, top, groups, keep);
     return check_launch("moe_route_sigmoid");
 }
 
@@ -331,8 +362,11 @@ int sllm_moe_silu_glu_scale(const void* u, const void* weights, void* y, int64_t
     const int64_t n = num_tokens * (int64_t)experts * ff;
     if (n == 0) return 0;
     SLLM_REQUIRE(u && y && weights, "moe_silu_glu_scale: null pointer");
-    SLLM_DISPATCH_DTYPE_F32(dtype, (moe_silu_glu_scale_kernel<T><<<(unsigned)cdiv(n, 256), 256, 0, (cudaStream_t)stream>>>(
-        (const T*)u, (const float*)weights, (T*)y, n, experts, ff)));
+    const bool quad = ff % 4 == 0 && (((uintptr_t)u | (uintptr_t)y) & 15) == 0;
+    SLLM_DISPATCH_DTYPE_F32(dtype, {
+        if (quad) moe_silu_glu_scale_kernel<T, 4><<<(unsigned)cdiv(n / 4, 256), 256, 0, (cudaStream_t)stream>>>((const T*)u, (const float*)weights, (T*)y, n, experts, ff);
+        else moe_silu_glu_scale_kernel<T, 1><<<(unsigned)cdiv(n, 256), 256, 0, (cudaStream_t)stream>>>((const T*)u, (const float*)weights, (T*)y, n, experts, ff);
+    });
     return check_launch("moe_silu_glu_scale");
 }
 

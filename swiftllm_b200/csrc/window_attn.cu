@@ -26,6 +26,11 @@
 //   shared_kv          the values are the un-normed keys: the cache row is [ inv (G fp32 values in 2 G elements, rounded up to 8) |
 //                      k (G x dk as projected, rounded up to 8) ], inv = 1 / sqrt(mean(k^2) + eps) of the head; the norm's weight
 //                      belongs to the query weights (q . (inv k w) = inv (q w) . k), so ONE staged tile serves as K and V
+//   krot > 0           shared_kv with rotation: a key head's part of the row is [ k as projected (dk) | its first krot entries times
+//                      the norm's weight, turned (not divided by the rms) ], and queries arrive as [ entries krot .. dk - 1 times the
+//                      key norm's weight | the turned entries ] (whole_norm_rope_store), so the score is inv q . (columns krot ..
+//                      krot + dk - 1 of the key part) and the value its first dk columns
+//   sinks              a learned number per head: the softmax's denominator also contains exp(sinks[h])
 // diff_combine: per token and head, o = a1 - lambda * a2 of two maps' outputs, o / sqrt(mean(o^2) + eps) * factor * sigmoid(gate).
 #include "mma_helpers.cuh"
 #include "typed_io.cuh"
@@ -56,6 +61,10 @@ __device__ __forceinline__ float rot_entry(const T* __restrict__ x, int j, int r
 // the shared_kv cache row: first element of the keys, elements per row
 __host__ __device__ __forceinline__ int shared_kv_key_offset(int G) { return (2 * G + 7) / 8 * 8; }
 __host__ __device__ __forceinline__ int shared_kv_row(int G, int dk) { return shared_kv_key_offset(G) + (G * dk + 7) / 8 * 8; }
+
+// bytes between the rows of a shared-memory tile of `cols` 16-bit entries (cols % 8 == 0): an odd number of 16-byte pieces, so that the
+// eight rows an ldmatrix reads fall into different bank groups
+__host__ __device__ __forceinline__ int tile_pitch(int cols) { const int c = cols >> 3; return (c + 1 + (c & 1)) * 16; }
 
 // What a query at position p sees, walked as ONE list of keys: entries 0 .. nk - 1 are the kept first positions that lie before the
 // window's start `lo`, the rest are lo, lo + 1, ..
@@ -136,6 +145,46 @@ __global__ void __launch_bounds__(128) shared_kv_store_kernel(
     }
 }
 
+// Queries and keys that are RMS-normed over their WHOLE projection (all heads together, weights qw [H * dk], kw [G * dk]) and then turned
+// on their first rot_dims entries, with the un-normed keys as values: one CTA per token writes the cache row (shared_kv with krot =
+// rot_dims, see the top of the file) and the queries in the order the attention kernels read them.
+template <typename T>
+__global__ void __launch_bounds__(256) whole_norm_rope_store_kernel(
+    const T* __restrict__ q, int64_t q_stride, const T* __restrict__ k, int64_t k_stride, const float* __restrict__ qw,
+    const float* __restrict__ kw, float eps, const float* __restrict__ cosb, const float* __restrict__ sinb,
+    const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, const int* __restrict__ block_table, int max_blocks_per_seq,
+    T* __restrict__ cache, int n_slots, int slot, int block_size, T* __restrict__ q_out, int H, int G, int dk, int rot, int halves) {
+    __shared__ float red[32];
+    const int64_t t = blockIdx.x;
+    const int pos = tok_pos[t];
+    const int blk = block_table[(int64_t)tok_seq[t] * max_blocks_per_seq + pos / block_size];
+    const int koff = shared_kv_key_offset(G), kw_cols = dk + rot, hq = H / G, pass = dk - rot;
+    T* dst = cache + (((int64_t)blk * n_slots + slot) * block_size + pos % block_size) * shared_kv_row(G, kw_cols);
+    const T* qr = q + t * q_stride;
+    const T* kr = k + t * k_stride;
+    const float* cs = cosb != nullptr ? cosb + t * (rot >> 1) : nullptr;
+    const float* sn = sinb != nullptr ? sinb + t * (rot >> 1) : nullptr;
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x; i < H * dk; i += blockDim.x) { const float v = ldf(qr + i); sq += v * v; }
+    for (int i = threadIdx.x; i < G * dk; i += blockDim.x) { const float v = ldf(kr + i); sk += v * v; }
+    const float qinv = 1.f / sqrtf(block_sum(sq, red) / (float)(H * dk) + eps);
+    const float kinv = 1.f / sqrtf(block_sum(sk, red) / (float)(G * dk) + eps);
+    for (int g = threadIdx.x; g < G; g += blockDim.x) reinterpret_cast<float*>(dst)[g] = kinv;
+    for (int i = threadIdx.x; i < G * kw_cols; i += blockDim.x) {
+        const int g = i / kw_cols, j = i - g * kw_cols;
+        const T* x = kr + g * dk;
+        if (j < dk) dst[koff + i] = x[j];
+        else stf(dst + koff + i, rot_entry(x, j - dk, rot, halves, cs, sn, 1.f, kw + g * dk));
+    }
+    T* qo = q_out + t * H * dk;
+    for (int i = threadIdx.x; i < H * dk; i += blockDim.x) {
+        const int h = i / dk, j = i - h * dk;
+        const T* x = qr + h * dk;
+        if (j < pass) stf(qo + i, ldf(x + rot + j) * qinv * qw[h * dk + rot + j] * kw[(h / hq) * dk + rot + j]);
+        else stf(qo + i, rot_entry(x, j - pass, rot, halves, cs, sn, qinv, qw + h * dk));
+    }
+}
+
 // ------------------------------------------------------------------ attention (fp32 CUDA cores)
 constexpr int WA_TILE = 32;        // keys per tile: one per lane in the score phase
 constexpr int WA_MAX_HPB = 8;      // query heads (warps) per CTA: heads of ONE key/value group, they share the staged tile
@@ -152,14 +201,14 @@ __global__ void __launch_bounds__(WA_MAX_HPB * 32) window_attn_kernel(
     int H, int G, int dk, int dv, int rot_dims, int window, float scale, float sink, int halves, float qk_norm_eps,
     float softcap, const float* __restrict__ vcos, const float* __restrict__ vsin, float out_scale,
     const float* __restrict__ qnorm_w, float prenorm_eps, int chunk, int vshare, int out_f32, const float* __restrict__ slopes,
-    int keep_first, int gate_per_head, int shared_kv) {
+    int keep_first, int gate_per_head, int shared_kv, int krot, const float* __restrict__ sinks) {
     extern __shared__ float smem[];
-    const int KP = dk + 1;
+    const int KW = dk + krot, KP = KW + 1;      // entries of a key head in the cache row; row pitch of the tile
     const int hpb = blockDim.x >> 5;
     float* qs = smem;                          // [hpb][dk]
-    float* kt = qs + hpb * dk;                 // [WA_TILE][dk + 1]
-    float* vt = kt + WA_TILE * KP;             // [WA_TILE][dv]
-    float* os = vt + WA_TILE * dv;             // [hpb][dv]: the head's output before it is turned back (vcos only)
+    float* kt = qs + hpb * dk;                 // [WA_TILE][KP]
+    float* vt = kt + WA_TILE * KP;             // [WA_TILE][dv] (not with shared_kv)
+    float* os = shared_kv ? vt : vt + WA_TILE * dv;      // [hpb][dv]: the head's output before it is turned back (vcos only)
     float* kinv = os + hpb * dv;               // [WA_TILE]: the keys' 1 / rms (shared_kv only)
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int64_t t = blockIdx.x;
@@ -167,7 +216,7 @@ __global__ void __launch_bounds__(WA_MAX_HPB * 32) window_attn_kernel(
     const int g = (blockIdx.y * hpb) / (H / G);
     const int pos = tok_pos[t];
     const int* bt = block_table + (int64_t)tok_seq[t] * max_blocks_per_seq;
-    const int row = shared_kv ? shared_kv_row(G, dk) : G * dk + (G / vshare) * dv;
+    const int row = shared_kv ? shared_kv_row(G, KW) : G * dk + (G / vshare) * dv;
     const int koff = shared_kv ? shared_kv_key_offset(G) : 0;
     const float slope = slopes != nullptr ? slopes[h] : 0.f;
 
@@ -193,7 +242,7 @@ __global__ void __launch_bounds__(WA_MAX_HPB * 32) window_attn_kernel(
     }
 
     // a sink takes part in the normalisation only: it enters the running (maximum, sum) as a key of score 0 without a value
-    float m = sink > 0.f ? 0.f : -INFINITY, l = sink;
+    float m = sinks != nullptr ? sinks[h] : sink > 0.f ? 0.f : -INFINITY, l = sinks != nullptr ? 1.f : sink;
     float acc[KR];
 #pragma unroll
     for (int k = 0; k < KR; k++) acc[k] = 0.f;
@@ -210,8 +259,8 @@ __global__ void __launch_bounds__(WA_MAX_HPB * 32) window_attn_kernel(
         for (int jj = warp; jj < nkeys; jj += hpb) {
             const int kp = key_position(base + jj, nk, lo);
             const T* src = cache + (((int64_t)bt[kp / block_size] * n_slots + slot) * block_size + kp % block_size) * row;
-            const T* ks = src + koff + g * dk;
-            for (int d = lane; d < dk; d += 32) kt[jj * KP + d] = ldf(ks + d);
+            const T* ks = src + koff + g * KW;
+            for (int d = lane; d < KW; d += 32) kt[jj * KP + d] = ldf(ks + d);
             if (shared_kv) {
                 if (lane == 0) kinv[jj] = reinterpret_cast<const float*>(src)[g];
                 continue;
@@ -223,7 +272,7 @@ __global__ void __launch_bounds__(WA_MAX_HPB * 32) window_attn_kernel(
         const float* qw = qs + warp * dk;
         float s = -INFINITY;
         if (lane < nkeys) {
-            const float* kr = kt + lane * KP;
+            const float* kr = kt + lane * KP + krot;
             float a = 0.f;
             for (int d = 0; d < dk; d++) a += qw[d] * kr[d];
             if (shared_kv) a *= kinv[lane];
@@ -311,12 +360,14 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
     int H, int G, int dk, int dv, int rot_dims, int window, float scale_log2, float sink, int halves, float qk_norm_eps,
     float softcap, const float* __restrict__ vcos, const float* __restrict__ vsin, float out_scale,
     const float* __restrict__ qnorm_w, float prenorm_eps, int chunk, int vshare, int out_f32, const float* __restrict__ slopes_,
-    int keep_first_, int gate_per_head_, int shared_kv_) {
+    int keep_first_, int gate_per_head_, int shared_kv_, int krot_, const float* __restrict__ sinks_) {
     const float* slopes = EXT ? slopes_ : nullptr;
-    const int keep_first = EXT ? keep_first_ : 0;
+    const float* sinks = EXT ? sinks_ : nullptr;
+    const int keep_first = EXT ? keep_first_ : 0, krot = EXT ? krot_ : 0;
     const bool gate_per_head = EXT && gate_per_head_, shared_kv = EXT && shared_kv_;
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    const int PQ = dk * 2 + 16, PK = dk * 2 + 16, PV = dv * 2 + 16;            // row pitches in bytes
+    const int KW = dk + krot;                                                  // entries of a key head in the cache row
+    const int PQ = dk * 2 + 16, PK = tile_pitch(KW), PV = shared_kv ? PK : dv * 2 + 16;      // row pitches in bytes
     unsigned char* Qs = smem_raw;                                              // [64][PQ]
     unsigned char* Ks = Qs + WT_ROWS * PQ;                                     // [2][64][PK]
     unsigned char* Vs = shared_kv ? Ks : Ks + 2 * WT_KEYS * PK;                // [2][64][PV] (shared_kv: the key tile itself)
@@ -326,9 +377,9 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
     const int hqp = 1 << hqp_log2;
     const int t_first = row0 + blockIdx.x * qt;
     const int ntok = min(qt, row0 + nrows - t_first);
-    const int row_elems = shared_kv ? shared_kv_row(G, dk) : G * dk + (G / vshare) * dv;
+    const int row_elems = shared_kv ? shared_kv_row(G, KW) : G * dk + (G / vshare) * dv;
     const int koff = shared_kv ? shared_kv_key_offset(G) : 0;
-    const int ck = dk >> 3, cv = dv >> 3;                                      // 16-byte chunks per key / value row
+    const int ck = KW >> 3, cv = dv >> 3;                                      // 16-byte chunks per key / value row
     const int half = rot_dims >> 1;
     // with a score cap: cap * tanh(s * scale / cap), then to base 2
     const float cap_in = softcap > 0.f ? scale_log2 * 0.6931471805599453f / softcap : 0.f;
@@ -360,7 +411,7 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
             if (ok) {
                 const int b = kp / block_size;
                 const int64_t rowi = ((int64_t)bt[b] * n_slots + slot) * block_size + (kp - b * block_size);
-                krow = cache + rowi * row_elems + koff + g * dk;
+                krow = cache + rowi * row_elems + koff + g * KW;
                 vrow = cache + rowi * row_elems + G * dk + (g / vshare) * dv;
                 if (shared_kv && part == 0) cp_async4(smem_u32(kinv + st * WT_KEYS + jj), cache + rowi * row_elems + 2 * g);
             } else if (shared_kv && part == 0) {
@@ -435,6 +486,11 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
         const float sl_b = slopes != nullptr && live_b ? slopes[g * hq + (r_b & (hqp - 1))] * 1.4426950408889634f : 0.f;
         float m_a = sink > 0.f ? 0.f : -INFINITY, m_b = m_a;
         float l_a = (lane & 3) == 0 ? sink : 0.f, l_b = l_a;
+        if (sinks != nullptr) {
+            if (live_a) m_a = sinks[g * hq + (r_a & (hqp - 1))] * 1.4426950408889634f;
+            if (live_b) m_b = sinks[g * hq + (r_b & (hqp - 1))] * 1.4426950408889634f;
+            l_a = l_b = (lane & 3) == 0 ? 1.f : 0.f;
+        }
         float o[DMAX / 8][4];
 #pragma unroll
         for (int nt = 0; nt < DMAX / 8; nt++) { o[nt][0] = o[nt][1] = o[nt][2] = o[nt][3] = 0.f; }
@@ -459,7 +515,7 @@ __global__ void __launch_bounds__(128, WT_KEYS == 32 ? 3 : 2) window_attn_mma_ke
 #pragma unroll
                         for (int np = 0; np < WT_KEYS / 16; np++) {
                             uint32_t b0, b1, b2, b3;
-                            ldmatrix_x4(smem_u32(Kt + (np * 16 + (lane >> 4) * 8 + (lane & 7)) * PK + (kk * 16 + ((lane >> 3) & 1) * 8) * 2),
+                            ldmatrix_x4(smem_u32(Kt + (np * 16 + (lane >> 4) * 8 + (lane & 7)) * PK + (krot + kk * 16 + ((lane >> 3) & 1) * 8) * 2),
                                         b0, b1, b2, b3);
                             mma_16816<T>(sc[2 * np], a, b0, b1);
                             mma_16816<T>(sc[2 * np + 1], a, b2, b3);
@@ -627,12 +683,14 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(
     int G, int dk, int dv, int rot_dims, int window, float scale_log2, float sink, int halves, float qk_norm_eps,
     float softcap, const float* __restrict__ vcos, const float* __restrict__ vsin, float out_scale,
     const float* __restrict__ qnorm_w, float prenorm_eps, int chunk, int vshare, int out_f32, const float* __restrict__ slopes_,
-    int keep_first_, int gate_per_head_, int shared_kv_) {
+    int keep_first_, int gate_per_head_, int shared_kv_, int krot_, const float* __restrict__ sinks_) {
     const float* slopes = EXT ? slopes_ : nullptr;
-    const int keep_first = EXT ? keep_first_ : 0;
+    const float* sinks = EXT ? sinks_ : nullptr;
+    const int keep_first = EXT ? keep_first_ : 0, krot = EXT ? krot_ : 0;
     const bool gate_per_head = EXT && gate_per_head_, shared_kv = EXT && shared_kv_;
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    const int PQ = dk * 2 + 16, PK = dk * 2 + 16, PV = dv * 2 + 16;            // row pitches in bytes
+    const int KW = dk + krot;                                                  // entries of a key head in the cache row
+    const int PQ = dk * 2 + 16, PK = tile_pitch(KW), PV = dv * 2 + 16;         // row pitches in bytes
     const int stage_bytes = KT * (PK + (shared_kv ? (int)sizeof(float) : PV));
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     unsigned char* Qs = smem_raw;                                              // [16][PQ]
@@ -642,7 +700,7 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(
     const int64_t t = row0 + blockIdx.x;
     const int pos = tok_pos[t];
     const int* bt = block_table + (int64_t)tok_seq[t] * max_blocks_per_seq;
-    const int row_elems = shared_kv ? shared_kv_row(G, dk) : G * dk + (G / vshare) * dv;
+    const int row_elems = shared_kv ? shared_kv_row(G, KW) : G * dk + (G / vshare) * dv;
     int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
     if (chunk > 0) lo = max(lo, pos / chunk * chunk);
     const int nk = EXT && window > 0 ? min(keep_first, lo) : 0;
@@ -653,8 +711,9 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(
     // LPR neighbouring lanes, one 16-byte piece of the key and of the value each
     constexpr int LPR = DMAX / 8, RPI = 32 / LPR;
     const int piece = lane % LPR;
-    const bool has_k = piece * 8 < dk, has_v = !shared_kv && piece * 8 < dv;
-    const int k_elem = (shared_kv ? shared_kv_key_offset(G) : 0) + g * dk + piece * 8, v_elem = G * dk + (g / vshare) * dv + piece * 8;
+    const bool has_k = piece * 8 < KW, has_v = !shared_kv && piece * 8 < dv;
+    const bool has_k2 = EXT && (piece + LPR) * 8 < KW;                         // key parts wider than LPR pieces (krot <= dk)
+    const int k_elem = (shared_kv ? shared_kv_key_offset(G) : 0) + g * KW + piece * 8, v_elem = G * dk + (g / vshare) * dv + piece * 8;
     auto find_row = [&](int it) -> int {
         const int e = it * KT + lane;
         if (lane >= KT || e >= total) return -1;
@@ -674,6 +733,7 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(
             const T* base = cache + (int64_t)max(src, 0) * row_elems;
             const int nb = src >= 0 ? 16 : 0;
             if (has_k) cp_async16(K + r * PK + piece * 16, base + k_elem, nb);
+            if (EXT && has_k2) cp_async16(K + r * PK + (piece + LPR) * 16, base + k_elem + LPR * 8, nb);
             if (has_v) cp_async16(V + r * PV + piece * 16, base + v_elem, nb);
         }
         cp_async_commit();
@@ -742,6 +802,10 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(
             const int hh = n * 8 + 2 * (lane & 3) + e;
             m[n][e] = sink > 0.f && warp == 0 ? 0.f : -INFINITY;
             l[n][e] = lane < 4 && warp == 0 ? sink : 0.f;
+            if (sinks != nullptr && warp == 0 && hh < hq) {
+                m[n][e] = sinks[g * hq + hh] * 1.4426950408889634f;
+                l[n][e] = lane < 4 ? 1.f : 0.f;
+            }
             sl[n][e] = slopes != nullptr && hh < hq ? slopes[g * hq + hh] * 1.4426950408889634f : 0.f;
         }
     float o[DMAX / 16][NH][4];
@@ -771,7 +835,7 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_attn_decode_kernel(
         for (int b = 0; b < KT / 16; b++)
 #pragma unroll
             for (int n = 0; n < NH; n++) { sc[b][n][0] = sc[b][n][1] = sc[b][n][2] = sc[b][n][3] = 0.f; }
-        const uint32_t k_addr = Kt + ((lane & 7) + ((lane >> 3) & 1) * 8) * PK + (lane >> 4) * 16;
+        const uint32_t k_addr = Kt + ((lane & 7) + ((lane >> 3) & 1) * 8) * PK + krot * 2 + (lane >> 4) * 16;
 #pragma unroll
         for (int kk = 0; kk < DMAX / 16; kk++) {
             if (kk * 16 < dk) {
@@ -964,7 +1028,7 @@ static int launch_window_attn_mma(const void* q, int64_t q_stride_t, const void*
                                   int dv, int rot_dims, int window, float scale, float sink, int halves, float qk_norm_eps,
                                   float softcap, const void* vcos, const void* vsin, float out_scale, const void* qnorm_w,
                                   float prenorm_eps, int chunk, int vshare, int out_f32, const void* slopes, int keep_first,
-                                  int gate_per_head, int shared_kv, cudaStream_t stream) {
+                                  int gate_per_head, int shared_kv, int krot, const void* sinks, cudaStream_t stream) {
     static unsigned long long attr_mask = 0;
     const int hq = H / G;
     int hqp_log2 = 0;
@@ -989,7 +1053,7 @@ static int launch_window_attn_mma(const void* q, int64_t q_stride_t, const void*
         const int64_t first = parts[k][0], count = parts[k][1];
         if (count <= 0) continue;
         if (k == 1 && hq <= 16) {
-            size_t smem = 16 * (size_t)(dk * 2 + 16) + WD_WARPS * WD_STAGES * (size_t)KT * ((dk * 2 + 16) + (shared_kv ? sizeof(float) : dv * 2 + 16));
+            size_t smem = 16 * (size_t)(dk * 2 + 16) + WD_WARPS * WD_STAGES * (size_t)KT * (tile_pitch(dk + krot) + (shared_kv ? sizeof(float) : dv * 2 + 16));
             const size_t merge = ((size_t)WD_WARPS * hq * dv + 2 * WD_WARPS * 16) * sizeof(float);
             if (smem < merge) smem = merge;
             kern_split<<<dim3((unsigned)count, (unsigned)G), WD_WARPS * 32, smem, stream>>>(
@@ -997,21 +1061,21 @@ static int launch_window_attn_mma(const void* q, int64_t q_stride_t, const void*
                 n_slots, slot, block_size, (const int*)block_table, max_blocks_per_seq, (const int*)tok_seq, (const int*)tok_pos,
                 (T*)out, out_stride_t, (int)first, hq, G, dk, dv, rot_dims, window, scale_log2, sink, halves, qk_norm_eps, softcap,
                 (const float*)vcos, (const float*)vsin, out_scale, (const float*)qnorm_w, prenorm_eps, chunk, vshare, out_f32,
-                (const float*)slopes, keep_first, gate_per_head, shared_kv);
+                (const float*)slopes, keep_first, gate_per_head, shared_kv, krot, (const float*)sinks);
             continue;
         }
         const int qt = k == 0 ? WT_ROWS >> hqp_log2 : 1;
         // measured on B200 (128 + 128 per head): prompt portions 24 - 26 % faster with 32-key tiles (three CTAs per SM instead of
         // two); decoded tokens faster with 64-key tiles at 512 CTAs (357 vs 385 us), with 32-key tiles at 2048 CTAs (950 vs 1220 us)
         const int keys = (k == 0 || count * G >= 7 * (int64_t)num_sms) ? 32 : 64;
-        size_t smem = (size_t)WT_ROWS * (dk * 2 + 16) + 2 * (size_t)keys * ((dk * 2 + 16) + (shared_kv ? sizeof(float) : dv * 2 + 16));
+        size_t smem = (size_t)WT_ROWS * (dk * 2 + 16) + 2 * (size_t)keys * (tile_pitch(dk + krot) + (shared_kv ? sizeof(float) : dv * 2 + 16));
         if (vcos != nullptr && smem < (size_t)WT_ROWS * dv * sizeof(float)) smem = (size_t)WT_ROWS * dv * sizeof(float);
         (keys == 32 ? kern_prompt : kern_decode)<<<dim3((unsigned)cdiv(count, qt), (unsigned)G), 128, smem, stream>>>(
             (const T*)q, q_stride_t, (const float*)cosb, (const float*)sinb, (const T*)gate, gate_stride_t, (const T*)cache,
             n_slots, slot, block_size, (const int*)block_table, max_blocks_per_seq, (const int*)tok_seq, (const int*)tok_pos,
             (T*)out, out_stride_t, (int)first, (int)count, qt, hq, hqp_log2, H, G, dk, dv, rot_dims, window, scale_log2, sink,
             halves, qk_norm_eps, softcap, (const float*)vcos, (const float*)vsin, out_scale, (const float*)qnorm_w, prenorm_eps,
-            chunk, vshare, out_f32, (const float*)slopes, keep_first, gate_per_head, shared_kv);
+            chunk, vshare, out_f32, (const float*)slopes, keep_first, gate_per_head, shared_kv, krot, (const float*)sinks);
     }
     return check_launch("window_attention (tensor cores)");
 }
@@ -1029,11 +1093,11 @@ static int launch_window_attn(const void* q, int64_t q_stride_t, const void* cos
                               int64_t out_stride_t, int64_t num_tokens, int H, int G, int dk, int dv, int rot_dims, int window,
                               float scale, float sink, int halves, float qk_norm_eps, float softcap, const void* vcos,
                               const void* vsin, float out_scale, const void* qnorm_w, float prenorm_eps, int chunk, int vshare,
-                              int out_f32, const void* slopes, int keep_first, int gate_per_head, int shared_kv,
-                              cudaStream_t stream) {
+                              int out_f32, const void* slopes, int keep_first, int gate_per_head, int shared_kv, int krot,
+                              const void* sinks, cudaStream_t stream) {
     static unsigned long long attr_mask = 0;
     const int hpb = heads_per_cta(H / G);
-    const size_t smem = ((size_t)hpb * dk + (size_t)WA_TILE * (dk + 1) + (size_t)WA_TILE * dv + (size_t)hpb * dv + WA_TILE) * sizeof(float);
+    const size_t smem = ((size_t)hpb * dk + (size_t)WA_TILE * (dk + krot + 1) + (shared_kv ? 0 : (size_t)WA_TILE * dv) + (size_t)hpb * dv + WA_TILE) * sizeof(float);
     SLLM_REQUIRE(smem <= 200 * 1024, "window_attention: head sizes %d / %d need %zu bytes of shared memory", dk, dv, smem);
     auto kern = window_attn_kernel<T, KR>;
     if (first_use_on_this_device(attr_mask))
@@ -1043,7 +1107,7 @@ static int launch_window_attn(const void* q, int64_t q_stride_t, const void* cos
         slot, block_size, (const int*)block_table, max_blocks_per_seq, (const int*)tok_seq, (const int*)tok_pos, (T*)out,
         out_stride_t, H, G, dk, dv, rot_dims, window, scale, sink, halves, qk_norm_eps, softcap, (const float*)vcos,
         (const float*)vsin, out_scale, (const float*)qnorm_w, prenorm_eps, chunk, vshare, out_f32, (const float*)slopes, keep_first,
-        gate_per_head, shared_kv);
+        gate_per_head, shared_kv, krot, (const float*)sinks);
     return check_launch("window_attention");
 }
 
@@ -1090,6 +1154,25 @@ int sllm_shared_kv_store(const void* k, int64_t k_row_stride, const void* tok_se
     return check_launch("shared_kv_store");
 }
 
+int sllm_whole_norm_rope_store(const void* q, int64_t q_row_stride, const void* k, int64_t k_row_stride, const void* q_norm_w,
+                               const void* k_norm_w, float eps, const void* cosb, const void* sinb, const void* tok_seq,
+                               const void* tok_pos, const void* block_table, int max_blocks_per_seq, void* cache, int n_slots, int slot,
+                               int block_size, void* q_out, int64_t num_tokens, int num_heads, int num_kv_heads, int dk, int rot_dims,
+                               int pair_halves, sllm_dtype_t dtype, sllm_stream_t stream) {
+    SLLM_REQUIRE(num_tokens >= 0 && num_heads > 0 && num_kv_heads > 0 && num_heads % num_kv_heads == 0 && dk > 0 && rot_dims >= 0 &&
+                 rot_dims <= dk && rot_dims % 2 == 0, "whole_norm_rope_store: bad shape (heads %d / %d, dk %d, rot_dims %d)", num_heads,
+                 num_kv_heads, dk, rot_dims);
+    SLLM_REQUIRE(slot >= 0 && slot < n_slots && block_size > 0, "whole_norm_rope_store: bad cache slot %d of %d", slot, n_slots);
+    if (num_tokens == 0) return 0;
+    SLLM_REQUIRE(q && k && q_norm_w && k_norm_w && tok_seq && tok_pos && block_table && cache && q_out && (rot_dims == 0 || (cosb && sinb)),
+                 "whole_norm_rope_store: null pointer");
+    SLLM_DISPATCH_DTYPE_F32(dtype, (whole_norm_rope_store_kernel<T><<<(unsigned)num_tokens, 256, 0, (cudaStream_t)stream>>>(
+        (const T*)q, q_row_stride, (const T*)k, k_row_stride, (const float*)q_norm_w, (const float*)k_norm_w, eps, (const float*)cosb,
+        (const float*)sinb, (const int*)tok_seq, (const int*)tok_pos, (const int*)block_table, max_blocks_per_seq, (T*)cache, n_slots,
+        slot, block_size, (T*)q_out, num_heads, num_kv_heads, dk, rot_dims, pair_halves)));
+    return check_launch("whole_norm_rope_store");
+}
+
 int sllm_window_attention_set_simt(int on) {
     const int old = g_window_simt ? 1 : 0;
     g_window_simt = on != 0;
@@ -1103,7 +1186,9 @@ int sllm_window_attention(const void* q, int64_t q_stride_t, const void* cosb, c
                           int dk, int dv, int rot_dims, int window, float scale, int sink, int pair_halves, float qk_norm_eps,
                           float softcap, const void* vcos, const void* vsin, float out_scale, const void* qnorm_w,
                           float prenorm_eps, int chunk, int vshare, int out_f32, const void* slopes, int keep_first,
-                          int gate_per_head, int shared_kv, sllm_dtype_t dtype, sllm_stream_t stream) {
+                          int gate_per_head, int shared_kv, int krot, const void* sinks, sllm_dtype_t dtype, sllm_stream_t stream) {
+    SLLM_REQUIRE(krot >= 0 && krot <= dk && (krot == 0 || shared_kv), "window_attention: %d turned entries beside shared keys of %d", krot, dk);
+    SLLM_REQUIRE(!(sink && sinks), "window_attention: a sink of score 0 or learned sinks, not both");
     SLLM_REQUIRE(keep_first >= 0 && (keep_first == 0 || chunk == 0), "window_attention: kept first positions (%d) exclude chunks",
                  keep_first);
     SLLM_REQUIRE(!shared_kv || (dk == dv && vshare == 1 && rot_dims == 0 && qk_norm_eps < 0.f && vcos == nullptr),
@@ -1124,15 +1209,15 @@ int sllm_window_attention(const void* q, int64_t q_stride_t, const void* cosb, c
     SLLM_REQUIRE(num_prefill_tokens >= 0 && num_prefill_tokens <= num_tokens, "window_attention: bad number of prompt rows");
     const float sinkw = sink ? 1.f : 0.f;
     const int hq = num_heads / num_kv_heads;
-    if (!g_window_simt && dtype != SLLM_F32 && dk % 16 == 0 && dv % 16 == 0 && dk <= 128 && dv <= 128 && hq <= WT_ROWS &&
+    if (!g_window_simt && dtype != SLLM_F32 && dk % 16 == 0 && dv % 16 == 0 && krot % 8 == 0 && dk <= 128 && dv <= 128 && hq <= WT_ROWS &&
         num_tokens < (1ll << 31)) {
 #define WA_MMA(DMAX, EXT)                                                                                                        \
     SLLM_DISPATCH_DTYPE(dtype, return (launch_window_attn_mma<T, DMAX, EXT>(q, q_stride_t, cosb, sinb, gate, gate_stride_t, cache,  \
         n_slots, slot, block_size, block_table, max_blocks_per_seq, tok_seq, tok_pos, out, out_stride_t, num_tokens,         \
         num_prefill_tokens, num_heads, num_kv_heads, dk, dv, rot_dims, window, scale, sinkw, pair_halves, qk_norm_eps, softcap, \
-        vcos, vsin, out_scale, qnorm_w, prenorm_eps, chunk, vshare, out_f32, slopes, keep_first, gate_per_head, shared_kv,        \
+        vcos, vsin, out_scale, qnorm_w, prenorm_eps, chunk, vshare, out_f32, slopes, keep_first, gate_per_head, shared_kv, krot, sinks, \
         (cudaStream_t)stream)))
-        const bool ext = slopes != nullptr || keep_first > 0 || gate_per_head || shared_kv;
+        const bool ext = slopes != nullptr || keep_first > 0 || gate_per_head || shared_kv || sinks != nullptr;
         const bool small = dk <= 64 && dv <= 64;
         if (ext) { if (small) { WA_MMA(64, true); } else { WA_MMA(128, true); } }
         else if (small) { WA_MMA(64, false); }
@@ -1143,7 +1228,7 @@ int sllm_window_attention(const void* q, int64_t q_stride_t, const void* cosb, c
     SLLM_DISPATCH_DTYPE_F32(dtype, return (launch_window_attn<T, KR>(q, q_stride_t, cosb, sinb, gate, gate_stride_t, cache,   \
         n_slots, slot, block_size, block_table, max_blocks_per_seq, tok_seq, tok_pos, out, out_stride_t, num_tokens,        \
         num_heads, num_kv_heads, dk, dv, rot_dims, window, scale, sinkw, pair_halves, qk_norm_eps, softcap, vcos, vsin,      \
-        out_scale, qnorm_w, prenorm_eps, chunk, vshare, out_f32, slopes, keep_first, gate_per_head, shared_kv,        \
+        out_scale, qnorm_w, prenorm_eps, chunk, vshare, out_f32, slopes, keep_first, gate_per_head, shared_kv, krot, sinks, \
         (cudaStream_t)stream)))
     if (dv <= 32) { WA_LAUNCH(1); }
     else if (dv <= 64) { WA_LAUNCH(2); }

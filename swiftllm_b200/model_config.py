@@ -63,6 +63,10 @@ LLAMA3_70B = dict(model_type="llama", num_hidden_layers=80, num_attention_heads=
                   rope_theta=500000.0, rms_norm_eps=1e-5, hidden_act="silu", rope_scaling=None)
 
 
+# first entry of a frequency-scaling tuple that follows the Llama 3.1 rule (bands of wavelengths, a blend by turns between them)
+WAVE_BANDS = "wave_bands"
+
+
 # ---------------------------------------------------------------- Bupozen
 @dataclasses.dataclass(frozen=True)
 class LatentAttentionSpec:
@@ -112,7 +116,8 @@ class WindowAttentionSpec:
     gate: bool = True               # element-wise sigmoid gate on the output (projection `g`)
     pair_halves: bool = False       # rotary pairs (i, i + rot_dims / 2) instead of (2i, 2i + 1)
     # (factor, original context, fast turns, slow turns): pairs that make fewer than `slow` turns over the original context are
-    # slowed by `factor`, pairs that make more than `fast` are kept, a linear ramp between; cos and sin get 0.1 ln(factor) + 1
+    # slowed by `factor`, pairs that make more than `fast` are kept, a linear ramp between; cos and sin get 0.1 ln(factor) + 1.
+    # (WAVE_BANDS, factor, original context, low, high): the Llama 3.1 rule (worker/token_model.py: rotary_frequencies)
     rot_scaling: Optional[tuple] = None
     qk_unit_norm: bool = False      # rotated queries and keys are divided by their root mean square over the head
     softcap: float = 0.0            # > 0: score <- softcap * tanh(score / softcap)
@@ -129,12 +134,15 @@ class WindowAttentionSpec:
     distance_bias: bool = False     # score <- score - 2^(-8 (h + 1) / heads) * (query position - key position)
     keep_first: int = 0             # with a window: the sequence's first positions stay visible
     gate_per_head: bool = False     # the output gate is one number per head
-    shared_kv: bool = False         # the values are the keys as projected (before their norm); no value projection, no rotation
+    shared_kv: bool = False         # the values are the keys as projected (before their norm); no value projection
+    whole_norm: bool = False        # queries / keys are RMS-normed over their whole projection (all heads together) BEFORE rotation
+    learned_sink: bool = False      # the softmax's denominator also contains exp(a learned number per head)
 
     @property
     def cache_width(self) -> int:
-        if self.shared_kv:          # [1 / rms of every key head, fp32 | keys as projected], both rounded up to 8 entries
-            return (2 * self.kv_heads + 7) // 8 * 8 + (self.kv_heads * self.dim + 7) // 8 * 8
+        # [1 / rms of every key head, fp32 | keys as projected (each with its turned entries)], both rounded up to 8 entries
+        if self.shared_kv:
+            return (2 * self.kv_heads + 7) // 8 * 8 + (self.kv_heads * (self.dim + self.rot_dims) + 7) // 8 * 8
         return self.kv_heads * (self.maps * self.dim + self.vdim)
 
     @property
@@ -168,6 +176,38 @@ class GatedLinearAttentionSpec:
     dim: int
     vdim: int
     tau: float
+    kv_from: Optional[int] = None
+    cache_width: int = 0
+
+
+@dataclasses.dataclass(frozen=True)
+class DeltaRuleSpec:
+    """Gated delta rule: q, k (kv_heads x dim) and v (heads x vdim) each through a causal convolution of `conv` taps and a SiLU; unit
+    queries and keys; per head S <- g S, u = beta (v - S^T k), S <- S + k u^T, out = S^T q (dim x vdim, fp32, one per sequence) with one
+    decay g and one beta per head and token; RMS-normed per head (weight of `vdim` entries), gated by silu(W_g h) and projected.  Head h
+    uses query / key head h // (heads // kv_heads).  No cache rows."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+    kv_from: Optional[int] = None
+    cache_width: int = 0
+
+    @property
+    def conv_channels(self) -> int:
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+
+@dataclasses.dataclass(frozen=True)
+class MatrixMemorySpec:
+    """Matrix memory with exponential input gate (mLSTM): per head S (dim x vdim), a normaliser (dim) and a running maximum (fp32, one set
+    per sequence); both gates' logits are capped by gate_cap tanh(. / gate_cap); the heads' outputs are RMS-normed (weight of heads x
+    vdim entries), gated by sigmoid(W_g h) and projected.  No cache rows."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
     kv_from: Optional[int] = None
     cache_width: int = 0
 
@@ -237,7 +277,8 @@ class FeedForwardSpec:
     limit: float = 0.0          # clamped_glu: bound of the gate (above) and of the up projection (both sides)
     # routing.  "top_softmax": softmax over the `top` largest logits.  "softmax_grouped": scores are a softmax over all experts,
     # only experts of the `keep` best of `groups` groups can be chosen, the chosen scores are renormalised and scaled.
-    # "sigmoid_bias": scores are sigmoids; the `top` largest score + bias (tensor `correction`) are chosen; weights are the scores.
+    # "sigmoid_bias": scores are sigmoids; the `top` largest score + bias (tensor `correction`) are chosen - among the `keep` best of
+    # `groups` groups, by the sum of a group's two largest -; weights are the scores.
     # "softmax_top": scores are a softmax over all experts; the `top` largest are chosen; weights are those scores as they are.
     routing: str = "top_softmax"
     groups: int = 1
@@ -628,3 +669,89 @@ class ZuzezenModelConfig:
     def load_from_model_path(model_path: str) -> "ZuzezenModelConfig":
         with open(os.path.join(model_path, "config.json"), "r", encoding="utf-8") as f:
             return ZuzezenModelConfig(json.load(f))
+
+
+# ---------------------------------------------------------------- Vorerax
+class VoreraxModelConfig:
+    """config.json of the Vorerax design: {"architecture": "Vorerax", "vocab", "width", "norm": {"eps"}, "residual_mult", "streams",
+    "embedding": {"scale", "bigram": {"buckets", "mul_prev", "mul_cur"}}, "layers": [{"type": "attention" | "delta" | "mlstm", "mixer":
+    {...}, "mlp": {"kind": "moe", "router": {"experts", "top", "groups": {"count", "keep"}}, "expert": {"ff"}} | null}, ...]}.
+    "attention": {"heads", "kv_heads", "dim", "vdim" (= dim), "scale", "mask": {"size"}, "rot": {"base", "dims", "scaling": {"factor",
+    "low", "high", "original"}}}; "delta": {"heads", "kv_heads", "dim", "vdim", "conv"}; "mlstm": {"heads", "dim", "vdim", "gate_cap"}.
+    Layers are sequential pre-norm blocks on `streams` residual streams (hyper-connections; without the key: one stream, plain residual
+    sum) whose outputs are multiplied by residual_mult.  Every size may differ from layer to layer."""
+    family = "vorerax"
+
+    def __init__(self, model_config: dict):
+        assert model_config.get("architecture") == "Vorerax", f"not a Vorerax config: {model_config.get('architecture')!r}"
+        self.raw = dict(model_config)
+        self.vocab_size = int(model_config["vocab"])
+        self.hidden_size = int(model_config["width"])
+        self.rms_norm_eps = float(model_config["norm"]["eps"])
+        self.residual_mult = float(model_config.get("residual_mult", 1.0))
+        self.hyper = bool(model_config.get("streams"))          # the streams' weights are tensors of the checkpoint
+        self.num_streams = int(model_config.get("streams") or 1)
+        assert 1 <= self.num_streams <= 16, "1 <= streams <= 16"
+        emb = model_config.get("embedding") or {}
+        self.embedding_scale = float(emb.get("scale", 1.0))
+        pair = emb.get("bigram")
+        self.pair_hash = PairHashSpec(int(pair["buckets"]), int(pair["mul_prev"]), int(pair["mul_cur"])) if pair else None
+        self.mixers, self.ffs = [], []
+        for i, layer in enumerate(model_config["layers"]):
+            m = layer["mixer"]
+            if layer["type"] == "attention":
+                rot, mask = m.get("rot") or {}, m.get("mask") or {}
+                sc = rot.get("scaling")
+                spec = WindowAttentionSpec(
+                    heads=int(m["heads"]), kv_heads=int(m.get("kv_heads") or m["heads"]), dim=int(m["dim"]), vdim=int(m.get("vdim", m["dim"])),
+                    window=int(mask.get("size", 0)), rot_base=float(rot.get("base", 10000.0)), rot_dims=int(rot.get("dims", 0)),
+                    scale=float(m["scale"]), sink=False, gate=True, pair_halves=True, gate_per_head=True, shared_kv=True, whole_norm=True,
+                    learned_sink=True,
+                    rot_scaling=(WAVE_BANDS, float(sc["factor"]), float(sc["original"]), float(sc["low"]), float(sc["high"])) if sc else None)
+                assert spec.heads % spec.kv_heads == 0, f"layer {i}: heads must be a multiple of kv_heads"
+                assert spec.vdim == spec.dim, f"layer {i}: the values are the keys, so vdim must equal dim"
+                assert spec.rot_dims % 2 == 0 and spec.rot_dims <= spec.dim, f"layer {i}: rot.dims must be even and <= dim"
+            elif layer["type"] == "delta":
+                spec = DeltaRuleSpec(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads") or m["heads"]), dim=int(m["dim"]),
+                                     vdim=int(m["vdim"]), conv=int(m["conv"]))
+                assert spec.heads % spec.kv_heads == 0, f"layer {i}: heads must be a multiple of kv_heads"
+                assert 1 <= spec.conv <= 8, f"layer {i}: 1 <= conv <= 8"
+            else:
+                assert layer["type"] == "mlstm", f"layer {i}: unknown mixer type {layer['type']!r}"
+                spec = MatrixMemorySpec(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), gate_cap=float(m["gate_cap"]))
+                assert spec.gate_cap > 0, f"layer {i}: gate_cap must be positive"
+            self.mixers.append(spec)
+            f = layer.get("mlp")
+            if f is None:
+                self.ffs.append(None)
+                continue
+            assert f["kind"] == "moe", f"layer {i}: unknown mlp kind {f['kind']!r}"
+            r = f["router"]
+            groups = r.get("groups") or {}
+            count = int(groups.get("count", 1))
+            ff = FeedForwardSpec("moe", int(f["expert"]["ff"]), int(r["experts"]), int(r["top"]), activation="silu_glu",
+                                 routing="sigmoid_bias", groups=count, keep=int(groups.get("keep", count)))
+            assert ff.experts % ff.groups == 0 and 0 < ff.keep <= ff.groups and 0 < ff.top <= ff.keep * (ff.experts // ff.groups), \
+                f"layer {i}: {ff.top} experts cannot be chosen from {ff.keep} of {ff.groups} groups of {ff.experts} experts"
+            self.ffs.append(ff)
+        self.num_layers = len(self.mixers)
+        self.cache_slot, self.cache_slots_per_width = _cache_geometry(self.mixers)
+
+    def get_kvslot_size(self, dtype: torch.dtype = torch.bfloat16) -> int:
+        """Bytes of cache one token occupies: one [1 / rms | keys with their turned entries] row per attention layer."""
+        return sum(w * n for w, n in self.cache_slots_per_width.items()) * dtype.itemsize
+
+    def get_state_size(self, dtype: torch.dtype = torch.bfloat16) -> int:
+        """Bytes of recurrent state one SEQUENCE occupies, whatever its length."""
+        n = 4 if self.pair_hash else 0
+        for s in self.mixers:
+            if isinstance(s, DeltaRuleSpec):
+                n += 4 * s.heads * s.dim * s.vdim + (s.conv - 1) * s.conv_channels * dtype.itemsize
+            elif isinstance(s, MatrixMemorySpec):
+                n += 4 * s.heads * (s.dim * s.vdim + s.dim + 1)
+        return n
+
+    @staticmethod
+    def load_from_model_path(model_path: str) -> "VoreraxModelConfig":
+        with open(os.path.join(model_path, "config.json"), "r", encoding="utf-8") as f:
+            return VoreraxModelConfig(json.load(f))

@@ -7,6 +7,7 @@
     buzarax     "architecture": "Buzarax"                   BuzaraxModelConfig     worker.buzarax_model.BuzaraxModel
     naforax     "architecture": "Naforax"                   NaforaxModelConfig     worker.naforax_model.NaforaxModel
     zuzezen     "architecture": "Zuzezen"                   ZuzezenModelConfig     worker.zuzezen_model.ZuzezenModel
+    vorerax     "architecture": "Vorerax"                   VoreraxModelConfig     worker.vorerax_model.VoreraxModel
 
 Every worker class has the same public surface (load_weights, profile_num_blocks, init_kvcache_and_swap, forward /
 forward_async with the prefill-chunks-then-decodes batch layout, free_seqs_resources), so schedulers, examples and
@@ -32,6 +33,8 @@ _FAMILIES = {
                 "swiftllm_b200.model_config:NaforaxModelConfig", "swiftllm_b200.worker.naforax_model:NaforaxModel"),
     "zuzezen": (lambda raw: raw.get("architecture") == "Zuzezen",
                 "swiftllm_b200.model_config:ZuzezenModelConfig", "swiftllm_b200.worker.zuzezen_model:ZuzezenModel"),
+    "vorerax": (lambda raw: raw.get("architecture") == "Vorerax",
+                "swiftllm_b200.model_config:VoreraxModelConfig", "swiftllm_b200.worker.vorerax_model:VoreraxModel"),
 }
 
 

@@ -8,19 +8,19 @@ from swiftllm_b200 import _lib
 
 
 def embed_pair_hash(tokens: torch.Tensor, infer_state, last_token: torch.Tensor, embed: torch.Tensor, pairs, buckets: int,
-                    mul_prev: int, mul_cur: int, x_copy: torch.Tensor = None, scale: float = 1.0):
-    """-> (x fp32 [T, W], h [T, W] in embed's dtype).  x = embed[token] * scale + pairs[hash(previous token, token)] (pairs may be None);
+                    mul_prev: int, mul_cur: int, x_copy: torch.Tensor = None, scale: float = 1.0, want_h: bool = True):
+    """-> (x fp32 [T, W], h [T, W] in embed's dtype, or None without want_h).  x = embed[token] * scale + pairs[hash(previous token, token)] (pairs may be None);
     the previous token of a step's first row comes from last_token[sequence row], which is then moved on to the step's last
     token.  x_copy (fp32 [T, W]) receives the same values."""
     _lib.require_device(embed)
     T, W = tokens.shape[0], embed.shape[1]
     assert tokens.dtype == torch.int32 and embed.is_contiguous() and (pairs is None or (pairs.is_contiguous() and pairs.dtype == embed.dtype))
     x = torch.empty((T, W), dtype=torch.float32, device=embed.device)
-    h = torch.empty((T, W), dtype=embed.dtype, device=embed.device)
+    h = torch.empty((T, W), dtype=embed.dtype, device=embed.device) if want_h else None
     st = infer_state
     _lib.check(_lib.lib().sllm_embed_pair_hash(
         tokens.data_ptr(), st.token_seq_ids.data_ptr(), st.token_positions.data_ptr(), _lib.ptr(last_token), embed.data_ptr(),
-        _lib.ptr(pairs), buckets, mul_prev, mul_cur, scale, x.data_ptr(), _lib.ptr(x_copy), h.data_ptr(), T, W,
+        _lib.ptr(pairs), buckets, mul_prev, mul_cur, scale, x.data_ptr(), _lib.ptr(x_copy), _lib.ptr(h), T, W,
         _lib.dtype_tag_f32(embed.dtype), _lib.stream()), "embed_pair_hash")
     if pairs is not None:
         _lib.check(_lib.lib().sllm_store_last_tokens(tokens.data_ptr(), st.seg_starts.data_ptr(), st.seq_ids.data_ptr(),
@@ -69,13 +69,15 @@ def tanh_cap_inplace(x: torch.Tensor, cap: float):
     _lib.check(_lib.lib().sllm_tanh_cap_inplace(x.data_ptr(), x.numel(), cap, _lib.dtype_tag_f32(x.dtype), _lib.stream()), "tanh_cap_inplace")
 
 
-def moe_route_sigmoid(logits: torch.Tensor, bias, top: int) -> torch.Tensor:
-    """logits fp32 [T, E] -> routing weights fp32 [T, E]: sigmoid scores at the `top` experts with the largest score + bias."""
+def moe_route_sigmoid(logits: torch.Tensor, bias, top: int, groups: int = 1, keep: int = 1) -> torch.Tensor:
+    """logits fp32 [T, E] -> routing weights fp32 [T, E]: sigmoid scores at the `top` experts with the largest score + bias; with
+    keep < groups only experts of the `keep` best of `groups` equal groups of neighbours (a group's score: the sum of its two largest
+    score + bias) can be chosen."""
     assert logits.dtype == torch.float32 and logits.is_contiguous() and (bias is None or bias.dtype == torch.float32)
     _lib.require_device(logits)
     w = torch.empty_like(logits)
     _lib.check(_lib.lib().sllm_moe_route_sigmoid(logits.data_ptr(), _lib.ptr(bias), w.data_ptr(), logits.shape[0], logits.shape[1], top,
-                                                 _lib.stream()), "moe_route_sigmoid")
+                                                 groups, keep, _lib.stream()), "moe_route_sigmoid")
     return w
 
 

@@ -5,7 +5,8 @@ Options (`AttnOptions`) that other designs switch on: rotary pairs as halves ins
 tanh cap on the scores, values that are stored turned by their position (the output is turned back), a factor on the output, an
 RMS norm with weight on every query / key head before it turns, a chunked mask, several key heads (score maps) per value head
 with fp32 output, and `diff_combine`, which turns two maps' outputs into one gated head; a bias on the distance, kept first
-positions beside the window, one gate per head, and values that are the un-normed keys (`shared_kv_store`)."""
+positions beside the window, one gate per head, values that are the un-normed keys (`shared_kv_store`; with rotation and a norm over the
+whole projection: `whole_norm_rope_store`), and a learned softmax sink per head."""
 import dataclasses
 import torch
 
@@ -30,14 +31,17 @@ class AttnOptions:
     # the values are the un-normed keys: a cache row is [1 / rms of every key head (fp32) | keys as projected], `shared_row_width`
     # entries wide; the weight of the keys' norm is part of q_norm
     shared_kv: bool = False
+    key_turned: int = 0             # with shared_kv: rows and queries as whole_norm_rope_store writes them for this many turned entries
+    sinks: object = None            # fp32 [H]: the softmax's denominator also contains exp(sinks[h])
 
 
 PLAIN = AttnOptions()
 
 
-def shared_row_width(kv_heads: int, dk: int) -> int:
-    """Entries of a cache row whose keys are also the values: 2 per key head for the fp32 norm, then the keys, both rounded up to 8."""
-    return (2 * kv_heads + 7) // 8 * 8 + (kv_heads * dk + 7) // 8 * 8
+def shared_row_width(kv_heads: int, dk: int, turned: int = 0) -> int:
+    """Entries of a cache row whose keys are also the values: 2 per key head for the fp32 norm, then the keys (each with its turned
+    entries), both rounded up to 8."""
+    return (2 * kv_heads + 7) // 8 * 8 + (kv_heads * (dk + turned) + 7) // 8 * 8
 
 
 def _stride0(x: torch.Tensor) -> int:
@@ -76,6 +80,26 @@ def shared_kv_store(k: torch.Tensor, cache: torch.Tensor, slot: int, block_table
         _lib.dtype_tag_f32(k.dtype), _lib.stream()), "shared_kv_store")
 
 
+def whole_norm_rope_store(q: torch.Tensor, k: torch.Tensor, q_norm: torch.Tensor, k_norm: torch.Tensor, eps: float, cos, sin,
+                          cache: torch.Tensor, slot: int, block_table: torch.Tensor, infer_state, heads: int, kv_heads: int, dk: int,
+                          rot_dims: int, pair_halves: bool) -> torch.Tensor:
+    """q [T, H * dk], k [T, G * dk] as projected (row-strided slices are fine) are RMS-normed over their whole rows (weights fp32
+    [H * dk], [G * dk]) and turned on the first rot_dims entries of every head.  Writes the tokens' cache rows [1 / rms | per key head:
+    k as projected, turned entries of k * weight] and returns the queries in the matching order (AttnOptions.key_turned = rot_dims)."""
+    T = q.shape[0]
+    assert q.stride(1) == 1 and k.stride(1) == 1 and q.shape == (T, heads * dk) and k.shape == (T, kv_heads * dk) and q.dtype == k.dtype
+    assert q_norm.dtype == k_norm.dtype == torch.float32 and q_norm.shape == (heads * dk,) and k_norm.shape == (kv_heads * dk,)
+    assert cache.is_contiguous() and cache.dtype == k.dtype and cache.shape[3] == shared_row_width(kv_heads, dk, rot_dims)
+    _lib.require_device(q)
+    out = torch.empty((T, heads * dk), dtype=q.dtype, device=q.device)
+    _lib.check(_lib.lib().sllm_whole_norm_rope_store(
+        q.data_ptr(), _stride0(q), k.data_ptr(), _stride0(k), q_norm.data_ptr(), k_norm.data_ptr(), eps, _lib.ptr(cos), _lib.ptr(sin),
+        infer_state.token_seq_ids.data_ptr(), infer_state.token_positions.data_ptr(), block_table.data_ptr(), block_table.shape[1],
+        cache.data_ptr(), cache.shape[1], slot, cache.shape[2], out.data_ptr(), T, heads, kv_heads, dk, rot_dims,
+        1 if pair_halves else 0, _lib.dtype_tag_f32(q.dtype), _lib.stream()), "whole_norm_rope_store")
+    return out
+
+
 def window_attention(q: torch.Tensor, gate, cache: torch.Tensor, slot: int, block_table: torch.Tensor, infer_state,
                      out: torch.Tensor, heads: int, kv_heads: int, dk: int, dv: int, rot_dims: int, window: int, scale: float,
                      sink: bool, cos: torch.Tensor, sin: torch.Tensor, opt: AttnOptions = PLAIN, vcos: torch.Tensor = None,
@@ -85,10 +109,11 @@ def window_attention(q: torch.Tensor, gate, cache: torch.Tensor, slot: int, bloc
     T = q.shape[0]
     assert q.stride(1) == 1 and out.stride(1) == 1 and q.shape == (T, heads * dk) and out.shape == (T, heads * dv)
     assert gate is None or (gate.shape == (T, heads if opt.gate_per_head else heads * dv) and gate.stride(1) == 1 and gate.dtype == q.dtype)
-    row = shared_row_width(kv_heads, dk) if opt.shared_kv else kv_heads * dk + kv_heads // opt.vshare * dv
+    row = shared_row_width(kv_heads, dk, opt.key_turned) if opt.shared_kv else kv_heads * dk + kv_heads // opt.vshare * dv
     assert cache.shape[3] == row and cache.dtype == q.dtype and (not opt.shared_kv or dk == dv)
     assert cache.shape[0] * cache.shape[1] * cache.shape[2] < 1 << 31       # rows are numbered in 32 bits
     assert opt.slopes is None or (opt.slopes.dtype == torch.float32 and opt.slopes.shape == (heads,))
+    assert opt.sinks is None or (opt.sinks.dtype == torch.float32 and opt.sinks.shape == (heads,) and not sink)
     assert out.dtype == (torch.float32 if opt.out_f32 else q.dtype)
     assert opt.q_norm is None or (opt.q_norm.dtype == torch.float32 and opt.q_norm.shape == (dk,))
     _lib.require_device(q)
@@ -99,7 +124,8 @@ def window_attention(q: torch.Tensor, gate, cache: torch.Tensor, slot: int, bloc
         min(T, max(0, int(getattr(infer_state, "num_prefill_tokens", T)))), heads, kv_heads, dk, dv, rot_dims, window, scale, 1 if sink else 0,
         1 if opt.pair_halves else 0, opt.qk_norm_eps, opt.softcap, _lib.ptr(vcos), _lib.ptr(vsin), opt.out_scale,
         _lib.ptr(opt.q_norm), opt.prenorm_eps, opt.chunk, opt.vshare, 1 if opt.out_f32 else 0,
-        _lib.ptr(opt.slopes), opt.keep_first, 1 if opt.gate_per_head else 0, 1 if opt.shared_kv else 0, _lib.dtype_tag_f32(q.dtype),
+        _lib.ptr(opt.slopes), opt.keep_first, 1 if opt.gate_per_head else 0, 1 if opt.shared_kv else 0,
+        opt.key_turned, _lib.ptr(opt.sinks), _lib.dtype_tag_f32(q.dtype),
         _lib.stream()),
         "window_attention")
 

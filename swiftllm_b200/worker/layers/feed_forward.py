@@ -1,7 +1,8 @@
 """Feed-forward sublayers: dense and mixture-of-experts with the squared-ReLU activation, a dense clamped gated linear unit, a
 dense GELU gated linear unit, a dense SiLU gated linear unit with biases, a mixture of clamped gated-linear-unit experts (group-limited routing with renormalised scores, or
 the plain softmax scores of the largest experts) with a shared expert that may have a per-token sigmoid weight, and a mixture of
-SiLU-gated experts routed by sigmoid scores with a bias that only takes part in the choice.
+SiLU-gated experts routed by sigmoid scores with a bias that only takes part in the choice (and, optionally, a limit to the best groups
+of experts).
 
 Every forward takes the sublayer's input `h` in the storage dtype and, optionally, the same input in fp32 (`x32`: designs whose
 sublayers read an fp32 stream hand it to the router, which then sees no rounding).
@@ -15,7 +16,7 @@ only matters once the step is compute-bound (a decode step streams every expert'
 tokens * top >= experts)."""
 import torch
 
-from swiftllm_b200.worker.kernels.linear import linear, linear_bias
+from swiftllm_b200.worker.kernels.linear import linear, linear_bias, linear_f32_out
 from swiftllm_b200.worker.kernels.parallel_block import (moe_clamped_glu_scale, moe_relu2_scale_inplace, moe_route,
                                                          moe_route_grouped, relu2_inplace)
 from swiftllm_b200.worker.kernels.sandwich_ops import gelu_glu, moe_route_softmax
@@ -110,17 +111,21 @@ class SiluGluFeedForward:
 
 class SiluGluMixtureOfExperts:
     """Experts y = silu(gate) * up -> down, no biases.  Routing: scores are sigmoids of fp32 router logits; the `top` experts with
-    the largest score + correction are chosen and weighted by their plain scores (not renormalised).  Dense formulation as above:
-    ONE [gate | up] GEMM over all experts, the activation kernel applies the routing weight (exact zeros for the others), ONE
-    down GEMM sums the chosen experts."""
+    the largest score + correction - among the `keep` best of `groups` groups, by the sum of a group's two largest - are chosen and
+    weighted by their plain scores (not renormalised).  Dense formulation as above: ONE [gate | up] GEMM over all experts, the
+    activation kernel applies the routing weight (exact zeros for the others), ONE down GEMM sums the chosen experts.  A router
+    stored in h's dtype reads h itself (fp32 accumulation, logits not rounded)."""
 
     def __init__(self, spec, weight):
         self.spec, self.weight = spec, weight
 
     def forward(self, h: torch.Tensor, x32=None) -> torch.Tensor:
         f, w = self.spec, self.weight
-        logits = linear(h.float() if x32 is None else x32, w.router)   # fp32 GEMM (TF32 stays off)
-        weights = moe_route_sigmoid(logits, w.correction, f.top)
+        if x32 is None and w.router.dtype == h.dtype:
+            logits = linear_f32_out(h, w.router)
+        else:
+            logits = linear(h.float() if x32 is None else x32, w.router)   # fp32 GEMM (TF32 stays off)
+        weights = moe_route_sigmoid(logits, w.correction, f.top, f.groups, f.keep)
         u = linear(h, w.up)                                     # [T, experts * 2 * ff]
         y = moe_silu_glu_scale(u, weights, f.experts, f.ff)
         return linear(y, w.down)

@@ -8,14 +8,17 @@ kernels.  `attend` is the part between the two GEMMs, for mixers that fuse their
 the cache holds the un-normed keys with their 1 / rms, and one staged tile serves the attention kernel as keys and values; scores
 carry a bias on the distance; the first positions of the sequence stay visible beside the window.
 
+`WholeNormAttentionMixer`: values that are the keys as projected, again, but queries and keys are normed over their whole projection and
+turn on a part of every head; the cache row holds the un-normed keys, their 1 / rms and the turned entries; a learned sink per head.
+
 `DifferentialAttentionMixer`: two score maps per head over the same values.  Every map is a query head of its own for the same two
 kernels (twice the heads, `vshare` = 2 key heads per value head, fp32 output); one more kernel subtracts the maps, normalises
 the head and applies the gate."""
 import torch
 
 from swiftllm_b200.worker.kernels.linear import linear, linear_bias
-from swiftllm_b200.worker.kernels.window_attn import (AttnOptions, diff_combine, shared_kv_store, window_attention,
-                                                      window_kv_store)
+from swiftllm_b200.worker.kernels.window_attn import (AttnOptions, diff_combine, shared_kv_store, whole_norm_rope_store,
+                                                      window_attention, window_kv_store)
 
 
 class WindowAttentionMixer:
@@ -94,6 +97,40 @@ class SharedKeyValueAttentionMixer:
             return linear(out.zero_(), w.o)
         cache = caches[self.cache_width]
         shared_kv_store(k, cache, self.cache_slot, block_table, st, m.kv_heads, m.dim, self.eps)
+        window_attention(q, gate, cache, self.cache_slot, block_table, st, out, m.heads, m.kv_heads, m.dim, m.dim, 0, m.window, m.scale,
+                         False, None, None, self.options)
+        return linear(out, w.o)
+
+
+class WholeNormAttentionMixer:
+    """ONE GEMM [q ; k ; gate] -> norms over the whole projections, rotation, queries in score order, cache store (one kernel) ->
+    attention (window, softmax with a learned sink, gate per head: one kernel) -> o GEMM.  A cached key is its projection (which is
+    the value), 1 / rms of the token's keys, and its turned entries with the norm's weight: the un-turned entries' weight is part of
+    the query (q . (k / rms * w) = (q * w) . k / rms)."""
+
+    def __init__(self, spec, weight, eps: float, cache_key):
+        assert spec.shared_kv and spec.whole_norm and spec.gate_per_head and spec.keep_first == 0 and spec.chunk == 0
+        self.spec, self.weight, self.eps = spec, weight, eps
+        self.cache_width, self.cache_slot = cache_key
+        self.options = AttnOptions(gate_per_head=True, shared_kv=True, key_turned=spec.rot_dims, sinks=weight.sink)
+
+    def register(self, model):
+        m = self.spec
+        model._register_rotary(m.rot_key, m.rot_base, m.rot_dims, m.rot_scaling)
+
+    def state_layout(self) -> dict:
+        return {}
+
+    def forward(self, h: torch.Tensor, caches: dict, block_table: torch.Tensor, states, st) -> torch.Tensor:
+        m, w = self.spec, self.weight
+        q, k, gate = torch.split(linear(h, w.in_proj), [m.heads * m.dim, m.kv_heads * m.dim, m.heads], dim=1)
+        out = torch.empty((h.shape[0], m.heads * m.dim), dtype=h.dtype, device=h.device)
+        if st.ignore_kvcache:
+            return linear(out.zero_(), w.o)
+        cos, sin = st.rotary[m.rot_key] if m.rot_dims > 0 else (None, None)
+        cache = caches[self.cache_width]
+        q = whole_norm_rope_store(q, k, w.q_norm, w.k_norm, self.eps, cos, sin, cache, self.cache_slot, block_table, st, m.heads,
+                                  m.kv_heads, m.dim, m.rot_dims, m.pair_halves)
         window_attention(q, gate, cache, self.cache_slot, block_table, st, out, m.heads, m.kv_heads, m.dim, m.dim, 0, m.window, m.scale,
                          False, None, None, self.options)
         return linear(out, w.o)

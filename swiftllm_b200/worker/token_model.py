@@ -3,8 +3,8 @@ position): the public surface of `LlamaModel` (worker/model.py), the paged cache
 recurrent state (worker/state_manager.py), the step's metadata and angle tables, and the CUDA-graph replay of pure-decode steps.
 A topology subclasses it (worker/parallel_block_model.py: parallel blocks; worker/buzarax_model.py: sequential blocks whose
 sublayer outputs are normalised, with recurrent mixers; worker/naforax_model.py: sequential blocks with norms on both sides of
-every sublayer, of which a range of layers runs several times; worker/zuzezen_model.py: the post-norm blocks with other mixers) and
-provides `_load_weights`, `_build_layers` and `_forward`.
+every sublayer, of which a range of layers runs several times; worker/zuzezen_model.py: the post-norm blocks with other mixers;
+worker/vorerax_model.py: pre-norm blocks on several residual streams) and provides `_load_weights`, `_build_layers` and `_forward`.
 
     Model(engine_config[, model_config]) -> load_weights() -> profile_num_blocks() -> init_kvcache_and_swap(num_blocks)
     forward(input_ids_list, seq_ids_list, decoding_seq_lens_list, ignore_kvcache=False, prefill_prefix_lens_list=None,
@@ -30,6 +30,7 @@ from typing import Callable, Optional
 import torch
 
 from swiftllm_b200.engine_config import EngineConfig
+from swiftllm_b200.model_config import WAVE_BANDS
 from swiftllm_b200.utils import GB
 from swiftllm_b200.worker.block_manager import BlockManager
 from swiftllm_b200.worker.state_manager import SequenceStateManager
@@ -44,10 +45,26 @@ def rotary_frequencies(base: float, dims: int, scaling: Optional[tuple] = None):
     """-> (frequency of every pair [dims / 2], factor on cos and sin).  Plain: base^(-2i/dims), factor 1.  With scaling =
     (factor, original context, fast, slow): the pair index at which a wavelength makes `turns` turns over the original context is
     d(turns) = dims ln(original / (2 pi turns)) / (2 ln base); pairs up to floor(d(fast)) keep their frequency, pairs from
-    ceil(d(slow)) on are slowed by `factor`, linearly blended between; cos and sin are multiplied by 0.1 ln(factor) + 1."""
+    ceil(d(slow)) on are slowed by `factor`, linearly blended between; cos and sin are multiplied by 0.1 ln(factor) + 1.  With scaling =
+    (WAVE_BANDS, factor, original context, low, high), the Llama 3.1 rule: a pair whose wavelength 2 pi / f is below original / high
+    keeps its frequency, above original / low it is slowed by `factor`, and between the two both are blended by
+    (original / wavelength - low) / (high - low); factor 1 on cos and sin."""
     f = [base ** (-2.0 * i / dims) for i in range(dims // 2)]
     if scaling is None:
         return f, 1.0
+    if scaling[0] == WAVE_BANDS:
+        _, factor, original, low, high = scaling
+        out = []
+        for fi in f:
+            turns = original * fi / (2.0 * math.pi)                     # original context / wavelength
+            if turns > high:
+                out.append(fi)
+            elif turns < low:
+                out.append(fi / factor)
+            else:
+                s = (turns - low) / (high - low)
+                out.append((1.0 - s) * fi / factor + s * fi)
+        return out, 1.0
     factor, original, fast, slow = scaling
 
     def pair_at(turns):

@@ -499,6 +499,107 @@ def load_zuzezen_weights(model_config, dtype: torch.dtype, model_path: Optional[
     return weight
 
 
+class StreamConnection:
+    """How a sublayer is tied to the residual streams, fp32: `read` (weights of the streams in its input), `mix` [from, to], `share` (of
+    its output, the residual multiplier included)."""
+
+    def __init__(self, read: torch.Tensor, mix: torch.Tensor, share: torch.Tensor):
+        self.read, self.mix, self.share = read, mix, share
+
+
+class VoreraxLayerWeight:
+    """One block on several residual streams.  Checkpoint names: `l<i>.{norm1, hc1.in, hc1.out, hc1.mix}` (and `norm2`, `hc2.*` with a
+    feed-forward; no `hc*` in a model without streams), and
+    mixer "attention": `l<i>.mix.{q, k, q.norm, k.norm, sink, g, o}`;
+    mixer "delta": `l<i>.mix.{q, q.conv, k, k.conv, v, v.conv, b, a, A_log, dt_bias, norm, g, o}`;
+    mixer "mlstm": `l<i>.mix.{q, k, v, g, norm, i, i.b, f, f.b, o}`;
+    feed-forward: `l<i>.mlp.{router, correction, e<k>.{gate, up, down}}`.
+    Fusions made at load time: every projection that reads the sublayer's input is one GEMM operand (`in_proj`: [q ; k ; g], [q ; k ; v ;
+    g]), the recurrences' small gate projections another whose result stays fp32 (`gate_proj`: [b ; a], [f ; i]); the three
+    convolutions are one (`conv`); `rate` = exp(A_log); the experts' [gate ; up] rows and down columns are concatenated expert by
+    expert; the residual multiplier is part of the streams' shares.  Norm weights, convolution taps, gate biases, sinks and the
+    streams' weights are fp32; the router is kept in the engine dtype (its logits are fp32 all the same)."""
+
+    def __init__(self, layer_id: int, model_config, dtype: torch.dtype):
+        self.layer_id, self.model_config, self.dtype = layer_id, model_config, dtype
+
+    def load_weights(self, getter: Callable, device):
+        from swiftllm_b200.model_config import DeltaRuleSpec, MatrixMemorySpec
+        c, i, f32 = self.model_config, self.layer_id, torch.float32
+        m, f, W, S = c.mixers[i], c.ffs[i], c.hidden_size, c.num_streams
+
+        def get(name, shape, dtype=None):
+            w = getter(f"l{i}.{name}", shape, dtype or self.dtype)
+            assert isinstance(w, torch.Tensor) and tuple(w.shape) == tuple(shape), f"l{i}.{name}: expected shape {tuple(shape)}"
+            return w.to(device=device, dtype=dtype or self.dtype).contiguous()
+
+        def connection(q):
+            if not c.hyper:
+                one = torch.ones((1,), dtype=f32, device=device)
+                return StreamConnection(one, one.view(1, 1), one * c.residual_mult)
+            return StreamConnection(get(f"hc{q}.in", (S,), f32), get(f"hc{q}.mix", (S, S), f32),
+                                    (get(f"hc{q}.out", (S,), f32) * c.residual_mult).contiguous())
+
+        self.norm1, self.conn1 = get("norm1", (W,), f32), connection(1)
+        H, dk, dv = m.heads, m.dim, m.vdim
+        if isinstance(m, DeltaRuleSpec):
+            G, K = m.kv_heads, m.conv
+            self.in_proj = torch.cat([get("mix.q", (G * dk, W)), get("mix.k", (G * dk, W)), get("mix.v", (H * dv, W)),
+                                      get("mix.g", (H * dv, W))], dim=0).contiguous()
+            self.conv = torch.cat([get("mix.q.conv", (G * dk, K), f32), get("mix.k.conv", (G * dk, K), f32),
+                                   get("mix.v.conv", (H * dv, K), f32)], dim=0).contiguous()
+            self.gate_proj = torch.cat([get("mix.b", (H, W)), get("mix.a", (H, W))], dim=0).contiguous()
+            self.decay_bias, self.rate = get("mix.dt_bias", (H,), f32), torch.exp(get("mix.A_log", (H,), f32)).contiguous()
+            self.head_norm = get("mix.norm", (dv,), f32)
+        elif isinstance(m, MatrixMemorySpec):
+            self.in_proj = torch.cat([get("mix.q", (H * dk, W)), get("mix.k", (H * dk, W)), get("mix.v", (H * dv, W)),
+                                      get("mix.g", (H * dv, W))], dim=0).contiguous()
+            self.gate_proj = torch.cat([get("mix.f", (H, W)), get("mix.i", (H, W))], dim=0).contiguous()
+            self.forget_bias, self.input_bias = get("mix.f.b", (H,), f32), get("mix.i.b", (H,), f32)
+            self.head_norm = get("mix.norm", (H * dv,), f32)
+        else:
+            G = m.kv_heads
+            self.in_proj = torch.cat([get("mix.q", (H * dk, W)), get("mix.k", (G * dk, W)), get("mix.g", (H, W))], dim=0).contiguous()
+            self.q_norm, self.k_norm = get("mix.q.norm", (H * dk,), f32), get("mix.k.norm", (G * dk,), f32)
+            self.sink = get("mix.sink", (H,), f32)
+        self.o = get("mix.o", (W, H * dv))
+        if f is None:
+            return
+        self.norm2, self.conn2 = get("norm2", (W,), f32), connection(2)
+        self.router, self.correction = get("mlp.router", (f.experts, W)), get("mlp.correction", (f.experts,), f32)
+        self.up = torch.cat([get(f"mlp.e{e}.{part}", (f.ff, W)) for e in range(f.experts) for part in ("gate", "up")], dim=0).contiguous()
+        self.down = torch.cat([get(f"mlp.e{e}.down", (W, f.ff)) for e in range(f.experts)], dim=1).contiguous()
+
+
+class VoreraxWeight:
+    def __init__(self, model_config, dtype: torch.dtype):
+        self.model_config, self.dtype = model_config, dtype
+        self.layers = [VoreraxLayerWeight(i, model_config, dtype) for i in range(model_config.num_layers)]
+
+    def load_weights(self, getter: Callable, device="cuda"):
+        c, f32 = self.model_config, torch.float32
+        vs = (c.vocab_size, c.hidden_size)
+        self.wte = getter("embed", vs, self.dtype).to(device=device, dtype=self.dtype).contiguous()
+        self.pairs = None
+        if c.pair_hash is not None:
+            self.pairs = getter("bigram", (c.pair_hash.buckets + 1, c.hidden_size), self.dtype).to(device=device, dtype=self.dtype).contiguous()
+        self.final_norm = getter("final.norm", (c.hidden_size,), f32).to(device=device, dtype=f32).contiguous()
+        self.final_read = torch.ones((c.num_streams,), dtype=f32, device=device)             # the model's output: the sum of the streams
+        self.lm_head = getter("head", vs, self.dtype).to(device=device, dtype=self.dtype).contiguous()
+        self.lm_head_sharded = False
+        for layer in self.layers:
+            layer.load_weights(getter, device)
+
+
+def load_vorerax_weights(model_config, dtype: torch.dtype, model_path: Optional[str], use_dummy: bool = False,
+                         getter: Optional[Callable] = None, device="cuda") -> VoreraxWeight:
+    if getter is None:
+        getter = dummy_getter(device) if use_dummy else checkpoint_getter(model_path, device)
+    weight = VoreraxWeight(model_config, dtype)
+    weight.load_weights(getter, device)
+    return weight
+
+
 # ---------------------------------------------------------------- getters
 def dummy_getter(device="cuda"):
     """weight.py:215-218: uniform(-1e-3, 1e-3), unseeded ("mainly for profiling")."""

@@ -12,9 +12,10 @@ from oracle import bupozen as O
 from oracle import buzarax as _buzarax
 from oracle import naforax as _naforax
 from oracle import rivudra as _rivudra
+from oracle import vorerax as _vorerax
 from oracle import zuzezen as _zuzezen
 
-_ORACLES = {"Bupozen": O, "Rivudra": _rivudra, "Buzarax": _buzarax, "Naforax": _naforax, "Zuzezen": _zuzezen}
+_ORACLES = {"Bupozen": O, "Rivudra": _rivudra, "Buzarax": _buzarax, "Naforax": _naforax, "Zuzezen": _zuzezen, "Vorerax": _vorerax}
 
 
 def oracle_of(cfg):

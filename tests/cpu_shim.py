@@ -304,8 +304,10 @@ def _window_attention(q, gate, cache, slot, block_table, st, out, heads, kv_head
         if opt and opt.shared_kv:
             off = (2 * kv_heads + 7) // 8 * 8
             inv = rows[:, :off].contiguous().view(torch.float32)[:, :kv_heads]
-            vg = rows[:, off:off + kv_heads * dk].float().view(-1, kv_heads, dk)
-            ks, vs = ((vg * inv[:, :, None]).repeat_interleave(rep, dim=1), vg.repeat_interleave(rep, dim=1))
+            kw = dk + opt.key_turned                          # per key head: the key, then its turned entries
+            kg = rows[:, off:off + kv_heads * kw].float().view(-1, kv_heads, kw)
+            vg, kg = kg[:, :, :dk], kg[:, :, opt.key_turned:]
+            ks, vs = ((kg * inv[:, :, None]).repeat_interleave(rep, dim=1), vg.repeat_interleave(rep, dim=1))
         else:
             rows = rows.float()
             ks = rows[:, :kv_heads * dk].view(-1, kv_heads, dk).repeat_interleave(rep, dim=1)     # [n, H, dk]
@@ -317,6 +319,8 @@ def _window_attention(q, gate, cache, slot, block_table, st, out, heads, kv_head
             sc = sc - opt.slopes[:, None] * (p - torch.tensor(seen, dtype=torch.float32))[None, :]
         if sink:
             sc = torch.cat([sc, torch.zeros(heads, 1)], dim=1)
+        if opt and opt.sinks is not None:
+            sc = torch.cat([sc, opt.sinks[:, None]], dim=1)
         pr = torch.softmax(sc, dim=-1)[:, :rows.shape[0]]
         o = torch.einsum("hn,nhd->hd", pr, vs)
         if vcos is not None:
@@ -326,6 +330,22 @@ def _window_attention(q, gate, cache, slot, block_table, st, out, heads, kv_head
             g = torch.sigmoid(gate[t].float())
             o = o * (g.repeat_interleave(dv) if opt and opt.gate_per_head else g)
         out[t] = o.to(out.dtype)
+
+
+def _whole_norm_rope_store(q, k, q_norm, k_norm, eps, cos, sin, cache, slot, block_table, st, heads, kv_heads, dk, rot_dims, pair_halves):
+    T, bs, off = q.shape[0], cache.shape[2], (2 * kv_heads + 7) // 8 * 8
+    kf = k.float()
+    inv = 1.0 / torch.sqrt((kf * kf).mean(-1) + eps)
+    turned = _rot_any((kf * k_norm).view(T, kv_heads, dk), cos, sin, rot_dims, pair_halves)[:, :, :rot_dims]
+    rows = torch.cat([kf.view(T, kv_heads, dk), turned], dim=2).reshape(T, -1)
+    for t, (sq, p) in enumerate(zip(st.token_seq_ids.tolist(), st.token_positions.tolist())):
+        row = cache[int(block_table[sq, p // bs]), slot, p % bs]
+        row[:off].view(torch.float32)[:kv_heads] = inv[t]
+        row[off:off + rows.shape[1]] = rows[t].to(cache.dtype)
+    qn = (_unit_rms(q.float(), eps) * q_norm).view(T, heads, dk)
+    plain = qn * k_norm.view(kv_heads, dk).repeat_interleave(heads // kv_heads, dim=0)
+    turned = _rot_any(qn, cos, sin, rot_dims, pair_halves)[:, :, :rot_dims]
+    return torch.cat([plain[:, :, rot_dims:], turned], dim=2).reshape(T, heads * dk).to(q.dtype)
 
 
 def _diff_combine(a, gate, out, heads, kv_heads, dv, lam, eps, factor):
@@ -454,7 +474,7 @@ def _segments(st):
     return [(sq, s[b], s[b + 1]) for b, sq in enumerate(st.seq_ids.tolist()) if s[b + 1] > s[b]]
 
 
-def _embed_pair_hash(tokens, st, last_token, embed, pairs, buckets, mul_prev, mul_cur, x_copy=None, scale=1.0):
+def _embed_pair_hash(tokens, st, last_token, embed, pairs, buckets, mul_prev, mul_cur, x_copy=None, scale=1.0, want_h=True):
     x = embed[tokens.long()].float() * scale
     if pairs is not None:
         pos = st.token_positions.tolist()
@@ -470,7 +490,7 @@ def _embed_pair_hash(tokens, st, last_token, embed, pairs, buckets, mul_prev, mu
             last_token[sq] = toks[hi - 1]
     if x_copy is not None:
         x_copy.copy_(x)
-    return x, x.to(embed.dtype)
+    return x, x.to(embed.dtype) if want_h else None
 
 
 def _postnorm_add_mix(x, y, gain, eps, h, history=None, slot=0, mix=None):
@@ -487,9 +507,15 @@ def _tanh_cap_inplace(x, cap):
     x.copy_(cap * torch.tanh(x / cap))
 
 
-def _moe_route_sigmoid(logits, bias, top):
+def _moe_route_sigmoid(logits, bias, top, groups=1, keep=1):
     s = torch.sigmoid(logits)
-    idx = torch.topk(s + (bias if bias is not None else 0.0), top, dim=-1).indices
+    c = s + (bias if bias is not None else 0.0)
+    if keep < groups:
+        per = c.view(c.shape[0], groups, -1)
+        score = per.topk(min(2, per.shape[2]), dim=2).values.sum(2)
+        stays = torch.zeros_like(score, dtype=torch.bool).scatter_(1, score.topk(keep, dim=1).indices, True)
+        c = per.masked_fill(~stays[:, :, None], float("-inf")).view(c.shape)
+    idx = torch.topk(c, top, dim=-1).indices
     return torch.zeros_like(s).scatter_(1, idx, s.gather(1, idx))
 
 
@@ -566,6 +592,73 @@ def _gla(q, k, v, z, bias, tau, norm_w, eps, gate, state, st, heads, dk, dv):
         state[sq] = S
     y = (_unit_rms(out, eps) * norm_w).reshape(T, heads * dv)
     return (y * torch.nn.functional.silu(gate.float())).to(q.dtype)
+
+
+def _delta_rule(q, k, v, decay_logits, beta_logits, decay_bias, rate, norm_w, eps, gate, state, st, heads, kv_heads, dk, dv):
+    T, rep = q.shape[0], heads // kv_heads
+
+    def unit(x):
+        x = x.float().view(T, kv_heads, dk)
+        return (x / torch.sqrt((x * x).sum(-1, keepdim=True) + 1e-6)).repeat_interleave(rep, dim=1)
+    qf, kf, vf = unit(q) * dk ** -0.5, unit(k), v.float().view(T, heads, dv)
+    g = torch.exp(-rate * torch.nn.functional.softplus(decay_logits + decay_bias))
+    beta = torch.sigmoid(beta_logits)
+    out = torch.zeros(T, heads, dv)
+    pos = st.token_positions.tolist()
+    for sq, lo, hi in _segments(st):
+        S = state[sq].clone() if pos[lo] > 0 else torch.zeros(heads, dk, dv)
+        for t in range(lo, hi):
+            S = g[t][:, None, None] * S
+            u = beta[t][:, None] * (vf[t] - torch.einsum("hkv,hk->hv", S, kf[t]))
+            S = S + kf[t][:, :, None] * u[:, None, :]
+            out[t] = torch.einsum("hkv,hk->hv", S, qf[t])
+        state[sq] = S
+    y = (_unit_rms(out, eps) * norm_w).reshape(T, heads * dv)
+    return (y * torch.nn.functional.silu(gate.float())).to(q.dtype)
+
+
+def _matrix_memory(q, k, v, forget_logits, input_logits, forget_bias, input_bias, cap, norm_w, eps, gate, state, norm_state, max_state,
+                   st, heads, dk, dv):
+    T = q.shape[0]
+    qf, kf, vf = q.float().view(T, heads, dk) * dk ** -0.5, k.float().view(T, heads, dk), v.float().view(T, heads, dv)
+    i = cap * torch.tanh((input_logits + input_bias) / cap)
+    f = torch.nn.functional.logsigmoid(cap * torch.tanh((forget_logits + forget_bias) / cap))
+    out = torch.zeros(T, heads, dv)
+    pos = st.token_positions.tolist()
+    for sq, lo, hi in _segments(st):
+        old = pos[lo] > 0
+        S = state[sq].clone() if old else torch.zeros(heads, dk, dv)
+        n = norm_state[sq].clone() if old else torch.zeros(heads, dk)
+        m = max_state[sq].clone() if old else torch.zeros(heads)
+        for t in range(lo, hi):
+            top = torch.maximum(f[t] + m, i[t])
+            keep, take = torch.exp(f[t] + m - top), torch.exp(i[t] - top)
+            m = top
+            S = keep[:, None, None] * S + take[:, None, None] * kf[t][:, :, None] * vf[t][:, None, :]
+            n = keep[:, None] * n + take[:, None] * kf[t]
+            den = torch.maximum((n * qf[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+            out[t] = torch.einsum("hkv,hk->hv", S, qf[t]) / den[:, None]
+        state[sq], norm_state[sq], max_state[sq] = S, n, m
+    y = _unit_rms(out, eps).reshape(T, heads * dv) * norm_w
+    return (y * torch.sigmoid(gate.float())).to(q.dtype)
+
+
+def _stream_mix_norm(x, streams, y=None, mix=None, share=None, x_out=None, read=None, norm_w=None, eps=0.0, out_dtype=None, rows=None):
+    xs = x[:, None].expand(-1, streams, -1) if x.dim() == 2 else x
+    if rows is not None:
+        xs = xs[rows.long()]
+    if y is not None:
+        yr = (y if rows is None else y[rows.long()]).float()
+        xs = torch.einsum("st,nsw->ntw", mix, xs) + share[None, :, None] * yr[:, None, :]
+    else:
+        xs = xs.clone()
+    h = None
+    if norm_w is not None:
+        h = (_unit_rms(torch.einsum("s,nsw->nw", read, xs), eps) * norm_w).to(out_dtype)
+    if x_out is not None:
+        assert rows is None
+        x_out.copy_(xs)
+    return h
 
 
 def _silu_glu(u):
@@ -674,6 +767,17 @@ _PATCHES = [
     ("swiftllm_b200.worker.zuzezen_model", "embed_pair_hash", _embed_pair_hash),
     ("swiftllm_b200.worker.zuzezen_model", "add_rmsnorm_f32", _add_rmsnorm_f32),
     ("swiftllm_b200.worker.zuzezen_model", "linear_f32_out", _linear_f32_out),
+    ("swiftllm_b200.worker.layers.feed_forward", "linear_f32_out", _linear_f32_out),
+    ("swiftllm_b200.worker.vorerax_model", "embed_pair_hash", _embed_pair_hash),
+    ("swiftllm_b200.worker.vorerax_model", "linear_f32_out", _linear_f32_out),
+    ("swiftllm_b200.worker.vorerax_model", "stream_mix_norm", _stream_mix_norm),
+    ("swiftllm_b200.worker.layers.hyper_block", "stream_mix_norm", _stream_mix_norm),
+    ("swiftllm_b200.worker.layers.window_attention", "whole_norm_rope_store", _whole_norm_rope_store),
+    ("swiftllm_b200.worker.layers.delta_rule", "delta_rule", _delta_rule),
+    ("swiftllm_b200.worker.layers.delta_rule", "short_conv", _short_conv),
+    ("swiftllm_b200.worker.layers.delta_rule", "linear_f32_out", _linear_f32_out),
+    ("swiftllm_b200.worker.layers.matrix_memory", "matrix_memory", _matrix_memory),
+    ("swiftllm_b200.worker.layers.matrix_memory", "linear_f32_out", _linear_f32_out),
     ("swiftllm_b200.worker.naforax_model", "embed_pair_hash", _embed_pair_hash),
     ("swiftllm_b200.worker.naforax_model", "tanh_cap_inplace", _tanh_cap_inplace),
     ("swiftllm_b200.worker.naforax_model", "group_norm_add_norm", _group_norm_add_norm),
