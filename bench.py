@@ -4,7 +4,7 @@
   python bench.py [--gpus N] [--steps K] [--warmup W]            # this implementation
   python bench.py --impl reference ...                            # CPU arm: torch-eager oracle port on host cores
   torchrun --nproc-per-node N bench.py --gpus N ...               # N > 1: tensor parallel (heads / FFN columns)
-  python bench.py --arch-compare all [--steps K] [--warmup W]     # NOT the headline: Bupozen / Rivudra / Buzarax / Naforax / Zuzezen workers beside the Llama worker
+  python bench.py --arch-compare all [--steps K] [--warmup W]     # NOT the headline: Bupozen / Rivudra / Buzarax / Naforax / Zuzezen / Vorerax workers beside the Llama worker
                                                                   # (prefill / decode tok/s, attention roofline), 1 GPU
 
 Workload: Llama-3-8B shapes, bf16, pure decode, batch 256, every sequence at
@@ -88,7 +88,7 @@ def parse():
     ap.add_argument("--no-live-traffic", action="store_true", help="skip the ncu DRAM-byte measurement of the decode kernel")
     ap.add_argument("--no-prefill", action="store_true")
     ap.add_argument("--arch-models", type=str, default="", metavar="NAMES",
-                    help="with --arch-compare: only these workers (comma-separated: bupozen, rivudra, buzarax, naforax, zuzezen, llama); default all")
+                    help="with --arch-compare: only these workers (comma-separated: bupozen, rivudra, buzarax, naforax, zuzezen, vorerax, llama); default all")
     ap.add_argument("--arch-compare", type=str, default="", metavar="SIZES",
                     help="instead of the headline workload: prefill and decode throughput of the Bupozen and Rivudra workers beside the "
                          "Llama worker at equal width / depth (random weights), with the attention kernels' roofline fractions; "
@@ -109,6 +109,7 @@ ARCH_SIZES = {
 }
 
 
+VORERAX_ROT, VORERAX_STREAMS = 32, 4      # turned entries of every attention head (of 128), residual streams
 NAFORAX_CHUNK = 8192      # positions per attention chunk: longer than the benchmark's sequences, so the mask is plain causal here
 
 
@@ -177,7 +178,20 @@ def _arch_models(sz, dtype, only=None):
     zuz = {"architecture": "Zuzezen", "vocab": sz["vocab"], "width": W, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
            "layers": [{"type": zuz_mixers[i % 4][0], "mixer": zuz_mixers[i % 4][1],
                        "mlp": None if i % 4 == 2 else {"kind": "dense", "ff": sz["ff"]}} for i in range(sz["layers"])]}
-    for name, raw in (("bupozen", bup), ("rivudra", riv), ("buzarax", buz), ("naforax", naf), ("zuzezen", zuz), ("llama", llama)):
+    # Vorerax: [windowed attention (heads / 4 key heads of W / H entries that are also the values, 32 of them turned, learned sinks)], [gated
+    # delta rule (128 x 128 state per head, heads / 2 query / key heads, 4 taps)], [matrix memory (128 x 128 per head)], [attention], each
+    # with 16 / 32 experts (4 groups, 2 kept); four residual streams
+    vatt = {"heads": H, "kv_heads": G, "dim": W // H, "vdim": W // H, "scale": (W // H) ** -0.5, "mask": {"size": sz["window"]},
+            "rot": {"base": 50000.0, "dims": VORERAX_ROT, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 4096}}}
+    vor_mixers = [("attention", vatt), ("delta", {"heads": H, "kv_heads": H // 2, "dim": 128, "vdim": 128, "conv": 4}),
+                  ("mlstm", {"heads": H, "dim": 128, "vdim": 128, "gate_cap": 12.0}), ("attention", vatt)]
+    vor_moe = {"kind": "moe", "expert": {"ff": sz["eff"]},
+               "router": {"experts": sz["experts"], "top": sz["top"], "groups": {"count": 4, "keep": 2}}}
+    vor = {"architecture": "Vorerax", "vocab": sz["vocab"], "width": W, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+           "streams": VORERAX_STREAMS, "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 1000003, "mul_cur": 31}},
+           "layers": [{"type": vor_mixers[i % 4][0], "mixer": vor_mixers[i % 4][1], "mlp": vor_moe} for i in range(sz["layers"])]}
+    for name, raw in (("bupozen", bup), ("rivudra", riv), ("buzarax", buz), ("naforax", naf), ("zuzezen", zuz), ("vorerax", vor),
+                      ("llama", llama)):
         if only and name not in only:
             continue
         ec = swiftllm_b200.EngineConfig(model_path="", use_dummy=False, block_size=16, gpu_mem_utilization=0.9, num_cpu_blocks=0,
@@ -237,7 +251,7 @@ def run_arch_compare(args):
             layers_pkg = "swiftllm_b200.worker.layers."
             if name in ("bupozen", "zuzezen"):
                 mod, attrs = importlib.import_module(layers_pkg + "latent_attention"), ["latent_attention"]
-            elif name in ("rivudra", "buzarax", "naforax"):
+            elif name in ("rivudra", "buzarax", "naforax", "vorerax"):
                 mod, attrs = importlib.import_module(layers_pkg + "window_attention"), ["window_attention"]
             else:
                 mod, attrs = importlib.import_module(layers_pkg + "transformer_layer"), ["prefill_attention", "paged_attention"]
@@ -260,6 +274,17 @@ def run_arch_compare(args):
                          "post_norms": (importlib.import_module(layers_pkg + "sequential_block"), "postnorm_add_mix"),
                          "silu_glu": (importlib.import_module(layers_pkg + "feed_forward"), "silu_glu"),
                          "sigmoid_gate": (importlib.import_module(layers_pkg + "latent_attention"), "sigmoid_gate_inplace")}
+            if name in ("rivudra", "buzarax", "vorerax"):
+                act = "moe_clamped_glu_scale" if name == "rivudra" else "moe_silu_glu_scale"
+                route = "moe_route_grouped" if name == "rivudra" else "moe_route_sigmoid"
+                ffm = importlib.import_module(layers_pkg + "feed_forward")
+                extra.update({"expert_activation": (ffm, act), "router": (ffm, route)})
+            if name == "vorerax":
+                extra.update({"delta_rule": (importlib.import_module(layers_pkg + "delta_rule"), "delta_rule"),
+                              "delta_conv": (importlib.import_module(layers_pkg + "delta_rule"), "short_conv"),
+                              "matrix_memory": (importlib.import_module(layers_pkg + "matrix_memory"), "matrix_memory"),
+                              "streams": (importlib.import_module(layers_pkg + "hyper_block"), "stream_mix_norm"),
+                              "qk_norm_store": (importlib.import_module(layers_pkg + "window_attention"), "whole_norm_rope_store")})
             extra_ms = {}
 
             def timed(fn, steps, warmup, after=None):
@@ -323,6 +348,7 @@ def run_arch_compare(args):
             model.free_seqs_resources(dids)
 
             L, H = sz["layers"], sz["heads"]
+            extra_roof = {}
             if name == "bupozen":
                 r, dr, Wn = 512, 64, sz["window"]
                 vis_pre = sum(min(p + 1, Wn) for p in range(prompt_len)) * n_prompts
@@ -414,6 +440,36 @@ def run_arch_compare(args):
                     "sigmoid_gate": (Ll * ntok * H * 128 * 4, Ll * ntok * H * 128 * 6, Ll * dec_batch * H * 128 * 4,
                                      Ll * dec_batch * H * 128 * 6),
                 }
+            elif name == "vorerax":
+                # attention layers 0 and 3 of every four: windowed; q + out + the rows once (prefill), the visible rows (decode)
+                kinds = [i % 4 for i in range(L)]
+                La, Ld, Lm = sum(k in (0, 3) for k in kinds), kinds.count(1), kinds.count(2)
+                Wn, D, nkv, Wd, rot, S = sz["window"], sz["width"] // H, max(1, H // 4), sz["width"], VORERAX_ROT, VORERAX_STREAMS
+                ntok, Hk = n_prompts * prompt_len, H // 2
+                vis_pre = sum(min(p + 1, Wn) for p in range(prompt_len)) * n_prompts
+                vis_dec = dec_batch * min(ctx + 1, Wn)
+                row = nkv * ((D + rot) * 2 + 4)
+                fl_pre, by_pre = La * vis_pre * H * D * 4, La * ntok * (2 * H * D * 2 + row)
+                fl_dec, by_dec = La * vis_dec * H * D * 4, La * vis_dec * row
+                # label -> (prefill FLOPs, bytes, decode FLOPs, bytes).  Delta rule: q, k, v, gate in and the product out (2 bytes), two fp32
+                # gate logits per head, three products with the state (6 dk dv FLOPs) per token and head; matrix memory: two products;
+                # decode reads and writes every sequence's fp32 state.  Convolution: 2 bytes in and out, decode adds the tail both ways.
+                # Streams: all streams both ways, the sublayer's output in, the next read out; the first write reads one stream, the
+                # last one writes none (and runs for the output rows only).
+                C4, nsub = (2 * Hk + H) * 128, 2 * L
+                dio, mio = Hk * 2 * 128 * 2 + H * (3 * 128 * 2 + 8), H * (5 * 128 * 2 + 8)
+                st_tok = Wd * ((nsub - 2) * (8 * S + 4) + 4 * S + 8)
+                extra_roof = {
+                    "delta_rule": (Ld * ntok * H * 6 * 128 * 128, Ld * ntok * dio, Ld * dec_batch * H * 6 * 128 * 128,
+                                   Ld * dec_batch * (H * 128 * 128 * 8 + dio)),
+                    "delta_conv": (Ld * ntok * C4 * 8, Ld * ntok * C4 * 4, Ld * dec_batch * C4 * 8, Ld * dec_batch * C4 * (4 + 12)),
+                    "matrix_memory": (Lm * ntok * H * 4 * 128 * 128, Lm * ntok * mio, Lm * dec_batch * H * 4 * 128 * 128,
+                                      Lm * dec_batch * (H * 128 * 129 * 8 + mio)),
+                    "streams": (nsub * ntok * Wd * S * S * 2, ntok * st_tok, nsub * dec_batch * Wd * S * S * 2,
+                                dec_batch * (st_tok + Wd * (4 * S + 4))),
+                    "qk_norm_store": (La * ntok * H * D * 8, La * ntok * (2 * H * D * 2 + nkv * D * 2 + row), La * dec_batch * H * D * 8,
+                                      La * dec_batch * (2 * H * D * 2 + nkv * D * 2 + row)),
+                }
             else:
                 D, nkv = sz["width"] // H, max(1, H // 4)
                 fl_pre = L * n_prompts * (prompt_len * (prompt_len + 1) // 2) * H * D * 4
@@ -424,8 +480,16 @@ def run_arch_compare(args):
             def roof(fl, by, ms):
                 t_min = max(fl / (peaks["bf16_tflops"] * 1e12), by / (peaks["hbm_gbs"] * 1e9)) * 1e3
                 return round(t_min / ms, 4) if ms > 0 else None
+            if name in ("rivudra", "buzarax", "vorerax"):
+                # experts' activation: the chosen experts' [gate | up] in, every expert's product out (zeros where it was not chosen);
+                # router: logits in, weights out (fp32)
+                Lff, E, F, shared = (L - 1 if name == "buzarax" else L), sz["experts"], sz["eff"], 1 if name == "rivudra" else 0
+                tok_p, tok_d = n_prompts * prompt_len, dec_batch
+                act_b = ((sz["top"] + shared) * 2 * F + (E + shared) * F) * 2
+                extra_roof["expert_activation"] = (Lff * tok_p * E * F * 8, Lff * tok_p * act_b, Lff * tok_d * E * F * 8, Lff * tok_d * act_b)
+                extra_roof["router"] = (Lff * tok_p * E * 8, Lff * tok_p * E * 8, Lff * tok_d * E * 8, Lff * tok_d * E * 8)
             other = {}
-            if name in ("buzarax", "naforax", "zuzezen"):
+            if extra_roof:
                 for k, (fp, bp, fd, bd) in extra_roof.items():
                     other[k] = {"prefill_ms": round(pre_extra.get(k, 0.0), 3), "decode_ms": round(dec_extra.get(k, 0.0), 3),
                                 "prefill_roofline_frac": roof(fp, bp, pre_extra.get(k, 0.0)),

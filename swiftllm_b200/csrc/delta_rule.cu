@@ -18,6 +18,6 @@ extern "C" int sllm_delta_rule(const void* q, int64_t q_stride, const void* k, i
     a.norm_w = (const float*)norm_w; a.norm_step = 0; a.state = (float*)state;
     a.seg_starts = (const int*)seg_starts; a.seq_ids = (const int*)seq_ids; a.tok_pos = (const int*)tok_pos;
     a.o_raw = (float*)workspace; a.out = out; a.out_stride = out_stride;
-    a.dtype = dtype; a.num_segs = num_segs; a.H = num_heads; a.G = num_kv_heads; a.dk = dk; a.dv = dv;
-    return hd_run<true>(a, num_tokens, num_prefill_tokens, num_prefill_segs, workspace_floats, (cudaStream_t)stream);
+    a.num_segs = num_segs; a.H = num_heads; a.G = num_kv_heads; a.dk = dk; a.dv = dv;
+    return hd_run<true>(a, dtype, num_tokens, num_prefill_tokens, num_prefill_segs, workspace_floats, (cudaStream_t)stream);
 }

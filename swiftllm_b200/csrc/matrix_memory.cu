@@ -20,6 +20,6 @@ extern "C" int sllm_matrix_memory(const void* q, int64_t q_stride, const void* k
     a.norm_w = (const float*)norm_w; a.norm_step = dv; a.state = (float*)state; a.nstate = (float*)norm_state; a.mstate = (float*)max_state;
     a.seg_starts = (const int*)seg_starts; a.seq_ids = (const int*)seq_ids; a.tok_pos = (const int*)tok_pos;
     a.o_raw = (float*)workspace; a.out = out; a.out_stride = out_stride;
-    a.dtype = dtype; a.num_segs = num_segs; a.H = num_heads; a.G = num_heads; a.dk = dk; a.dv = dv;
-    return hd_run<false>(a, num_tokens, num_prefill_tokens, num_prefill_segs, workspace_floats, (cudaStream_t)stream);
+    a.num_segs = num_segs; a.H = num_heads; a.G = num_heads; a.dk = dk; a.dv = dv;
+    return hd_run<false>(a, dtype, num_tokens, num_prefill_tokens, num_prefill_segs, workspace_floats, (cudaStream_t)stream);
 }

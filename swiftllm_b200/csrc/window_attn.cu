@@ -146,42 +146,90 @@ __global__ void __launch_bounds__(128) shared_kv_store_kernel(
 }
 
 // Queries and keys that are RMS-normed over their WHOLE projection (all heads together, weights qw [H * dk], kw [G * dk]) and then turned
-// on their first rot_dims entries, with the un-normed keys as values: one CTA per token writes the cache row (shared_kv with krot =
-// rot_dims, see the top of the file) and the queries in the order the attention kernels read them.
-template <typename T>
+// on their first rot entries, with the un-normed keys as values: one CTA per token writes the cache row (shared_kv with krot = rot, see
+// the top of the file) and the queries in the order the attention kernels read them.  Both rows wait in shared memory as fp32
+// ((H + G) dk floats) between the sums and the writes; then a warp takes a head at a time.  VEC: eight entries a load (rows aligned,
+// H dk and G dk multiples of 8) and two a store (dk even).
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) whole_norm_rope_store_kernel(
     const T* __restrict__ q, int64_t q_stride, const T* __restrict__ k, int64_t k_stride, const float* __restrict__ qw,
     const float* __restrict__ kw, float eps, const float* __restrict__ cosb, const float* __restrict__ sinb,
     const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, const int* __restrict__ block_table, int max_blocks_per_seq,
     T* __restrict__ cache, int n_slots, int slot, int block_size, T* __restrict__ q_out, int H, int G, int dk, int rot, int halves) {
+    extern __shared__ __align__(16) float smem[];
     __shared__ float red[32];
+    constexpr int N = VEC ? 2 : 1;
     const int64_t t = blockIdx.x;
+    float* qs = smem;                          // [H * dk]
+    float* ks = qs + H * dk;                   // [G * dk]
     const int pos = tok_pos[t];
     const int blk = block_table[(int64_t)tok_seq[t] * max_blocks_per_seq + pos / block_size];
     const int koff = shared_kv_key_offset(G), kw_cols = dk + rot, hq = H / G, pass = dk - rot;
     T* dst = cache + (((int64_t)blk * n_slots + slot) * block_size + pos % block_size) * shared_kv_row(G, kw_cols);
-    const T* qr = q + t * q_stride;
-    const T* kr = k + t * k_stride;
     const float* cs = cosb != nullptr ? cosb + t * (rot >> 1) : nullptr;
     const float* sn = sinb != nullptr ? sinb + t * (rot >> 1) : nullptr;
-    float sq = 0.f, sk = 0.f;
-    for (int i = threadIdx.x; i < H * dk; i += blockDim.x) { const float v = ldf(qr + i); sq += v * v; }
-    for (int i = threadIdx.x; i < G * dk; i += blockDim.x) { const float v = ldf(kr + i); sk += v * v; }
+    auto stage = [&](const T* src, float* to, int n) {
+        float ss = 0.f;
+        if constexpr (VEC) {
+            constexpr int E = 16 / sizeof(T);
+            for (int i = threadIdx.x * E; i < n; i += blockDim.x * E) {
+                const uint4 u = *reinterpret_cast<const uint4*>(src + i);
+                const T* e = reinterpret_cast<const T*>(&u);
+#pragma unroll
+                for (int j = 0; j < E; j += 4) {
+                    const float4 v = make_float4(ldf(e + j), ldf(e + j + 1), ldf(e + j + 2), ldf(e + j + 3));
+                    *reinterpret_cast<float4*>(to + i + j) = v;
+                    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+                }
+            }
+        } else {
+            for (int i = threadIdx.x; i < n; i += blockDim.x) { const float v = ldf(src + i); to[i] = v; ss += v * v; }
+        }
+        return ss;
+    };
+    const float sq = stage(q + t * q_stride, qs, H * dk), sk = stage(k + t * k_stride, ks, G * dk);
     const float qinv = 1.f / sqrtf(block_sum(sq, red) / (float)(H * dk) + eps);
-    const float kinv = 1.f / sqrtf(block_sum(sk, red) / (float)(G * dk) + eps);
+    const float kinv = 1.f / sqrtf(block_sum(sk, red) / (float)(G * dk) + eps);          // (both rows are staged)
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5, half = rot >> 1;
     for (int g = threadIdx.x; g < G; g += blockDim.x) reinterpret_cast<float*>(dst)[g] = kinv;
-    for (int i = threadIdx.x; i < G * kw_cols; i += blockDim.x) {
-        const int g = i / kw_cols, j = i - g * kw_cols;
-        const T* x = kr + g * dk;
-        if (j < dk) dst[koff + i] = x[j];
-        else stf(dst + koff + i, rot_entry(x, j - dk, rot, halves, cs, sn, 1.f, kw + g * dk));
-    }
-    T* qo = q_out + t * H * dk;
-    for (int i = threadIdx.x; i < H * dk; i += blockDim.x) {
-        const int h = i / dk, j = i - h * dk;
-        const T* x = qr + h * dk;
-        if (j < pass) stf(qo + i, ldf(x + rot + j) * qinv * qw[h * dk + rot + j] * kw[(h / hq) * dk + rot + j]);
-        else stf(qo + i, rot_entry(x, j - pass, rot, halves, cs, sn, qinv, qw + h * dk));
+    auto put = [&](T* to, const float* v) {                              // N neighbouring entries
+        if constexpr (VEC) {
+            struct alignas(2 * sizeof(T)) Pair { T e[2]; } x;
+            stf(x.e, v[0]); stf(x.e + 1, v[1]);
+            *reinterpret_cast<Pair*>(to) = x;
+        } else {
+            stf(to, v[0]);
+        }
+    };
+    // the turned entries of a head x (weights w): pair i of `half`
+    auto turn = [&](T* to, const float* x, const float* w, float inv) {
+        for (int i = lane; i < half; i += 32) {
+            const int ia = halves ? i : 2 * i, ib = halves ? i + half : 2 * i + 1;
+            const float a = x[ia] * inv * w[ia], b = x[ib] * inv * w[ib];
+            stf(to + ia, a * cs[i] - b * sn[i]);
+            stf(to + ib, b * cs[i] + a * sn[i]);
+        }
+    };
+    for (int unit = warp; unit < H + G; unit += nwarps) {
+        if (unit < G) {
+            const int g = unit;
+            T* to = dst + koff + g * kw_cols;
+            for (int j = lane * N; j < dk; j += 32 * N) put(to + j, ks + g * dk + j);
+            turn(to + dk, ks + g * dk, kw + g * dk, 1.f);
+        } else {
+            const int h = unit - G, g = h / hq;
+            T* to = q_out + (t * H + h) * dk;
+            const float* x = qs + h * dk + rot;
+            const float* w = qw + h * dk + rot;
+            const float* wk = kw + g * dk + rot;
+            for (int j = lane * N; j < pass; j += 32 * N) {
+                float v[N];
+#pragma unroll
+                for (int e = 0; e < N; e++) v[e] = x[j + e] * qinv * w[j + e] * wk[j + e];
+                put(to + j, v);
+            }
+            turn(to + pass, qs + h * dk, qw + h * dk, qinv);
+        }
     }
 }
 
@@ -1166,10 +1214,24 @@ int sllm_whole_norm_rope_store(const void* q, int64_t q_row_stride, const void* 
     if (num_tokens == 0) return 0;
     SLLM_REQUIRE(q && k && q_norm_w && k_norm_w && tok_seq && tok_pos && block_table && cache && q_out && (rot_dims == 0 || (cosb && sinb)),
                  "whole_norm_rope_store: null pointer");
-    SLLM_DISPATCH_DTYPE_F32(dtype, (whole_norm_rope_store_kernel<T><<<(unsigned)num_tokens, 256, 0, (cudaStream_t)stream>>>(
-        (const T*)q, q_row_stride, (const T*)k, k_row_stride, (const float*)q_norm_w, (const float*)k_norm_w, eps, (const float*)cosb,
-        (const float*)sinb, (const int*)tok_seq, (const int*)tok_pos, (const int*)block_table, max_blocks_per_seq, (T*)cache, n_slots,
-        slot, block_size, (T*)q_out, num_heads, num_kv_heads, dk, rot_dims, pair_halves)));
+    const size_t smem = (size_t)(num_heads + num_kv_heads) * dk * sizeof(float);
+    SLLM_REQUIRE(smem <= 200 * 1024, "whole_norm_rope_store: %d + %d heads of %d entries do not fit in shared memory", num_heads,
+                 num_kv_heads, dk);
+    const int per = dtype == SLLM_F32 ? 4 : 8;
+    const bool vec = dk % 2 == 0 && (num_heads * dk) % per == 0 && (num_kv_heads * dk) % per == 0 && q_row_stride % per == 0 &&
+                     k_row_stride % per == 0 && (((uintptr_t)q | (uintptr_t)k | (uintptr_t)q_out | (uintptr_t)cache) & 15) == 0;
+    SLLM_DISPATCH_DTYPE_F32(dtype, {
+        static unsigned long long attr_mask = 0;
+        if (first_use_on_this_device(attr_mask)) {
+            cudaFuncSetAttribute(whole_norm_rope_store_kernel<T, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+            cudaFuncSetAttribute(whole_norm_rope_store_kernel<T, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+        }
+        (vec ? whole_norm_rope_store_kernel<T, true> : whole_norm_rope_store_kernel<T, false>)<<<(unsigned)num_tokens, 256, smem,
+                                                                                             (cudaStream_t)stream>>>(
+            (const T*)q, q_row_stride, (const T*)k, k_row_stride, (const float*)q_norm_w, (const float*)k_norm_w, eps, (const float*)cosb,
+            (const float*)sinb, (const int*)tok_seq, (const int*)tok_pos, (const int*)block_table, max_blocks_per_seq, (T*)cache, n_slots,
+            slot, block_size, (T*)q_out, num_heads, num_kv_heads, dk, rot_dims, pair_halves);
+    });
     return check_launch("whole_norm_rope_store");
 }
 

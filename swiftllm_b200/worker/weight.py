@@ -618,7 +618,7 @@ def synthetic_getter(seed: int = 0, std: float = 0.02, device="cuda", norm_offse
         g = torch.Generator(device=device)
         g.manual_seed((seed * 1000003 + zlib.crc32(key.encode())) & 0x7FFFFFFF)
         t = torch.randn(shape, generator=g, device=device, dtype=torch.float32) * std
-        if key.endswith(("norm.weight", "layernorm.weight", ".norm", ".norm1")):
+        if key.endswith(("norm.weight", "layernorm.weight", ".norm", ".norm1", ".norm2")):
             t += norm_offset
         return t.to(dtype)
     return get

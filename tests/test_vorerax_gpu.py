@@ -337,7 +337,7 @@ def test_bfloat16_worker_close_to_fp32_oracle():
     """bf16 projections / cache, fp32 streams, norms, attention weights, gates and states: the logits stay within bf16 rounding of the
     fp32 oracle on the same weights, and do not depend on how the prompt was cut beyond that.  The corrections are further apart than
     the scores, so that rounding cannot turn a choice of experts."""
-    for cfg, n, cuts, bs, nb in ((C.full_config(eps=1e-2), 33, [5, 2, 1, 1, 24], 4, 40), (_tc_config(), 150, [61, 4, 64, 2, 1, 1, 17], 8, 60)):
+    for cfg, n, cuts, bs, nb in ((C.full_config(eps=1e-2, mult=0.1), 33, [5, 2, 1, 1, 24], 4, 40), (_tc_config(), 150, [61, 4, 64, 2, 1, 1, 17], 8, 60)):
         t = O.random_tensors(cfg, seed=11)
         for name in t:
             if name.endswith("correction"):
@@ -347,7 +347,7 @@ def test_bfloat16_worker_close_to_fp32_oracle():
         m = B.make_worker(_make, cfg, t, dtype="bfloat16", block_size=bs, num_blocks=nb)
         whole = B.run_portions(m, toks, 0, [n])[-40:]
         cut = B.run_portions(m, toks, 1, cuts)[-40:]
-        assert B.rel_err(whole, ref) < 5e-2 and B.rel_err(cut, ref) < 5e-2 and B.rel_err(cut, whole) < 4e-2
+        assert B.rel_err(whole, ref) < 2e-2 and B.rel_err(cut, ref) < 2e-2 and B.rel_err(cut, whole) < 2e-2
 
 
 def test_cuda_graph_decode_matches_eager():
