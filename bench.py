@@ -279,6 +279,8 @@ def run_arch_compare(args):
                 route = "moe_route_grouped" if name == "rivudra" else "moe_route_sigmoid"
                 ffm = importlib.import_module(layers_pkg + "feed_forward")
                 extra.update({"expert_activation": (ffm, act), "router": (ffm, route)})
+            if name == "rivudra":
+                extra["kv_store"] = (importlib.import_module(layers_pkg + "window_attention"), "window_kv_store")
             if name == "vorerax":
                 extra.update({"delta_rule": (importlib.import_module(layers_pkg + "delta_rule"), "delta_rule"),
                               "delta_conv": (importlib.import_module(layers_pkg + "delta_rule"), "short_conv"),
@@ -365,6 +367,9 @@ def run_arch_compare(args):
                 vis_dec = dec_batch * min(ctx + 1, Wn)
                 fl_dec = L * vis_dec * H * D * 4
                 by_dec = L * vis_dec * 2 * nkv * D * 2
+                # keys and values in, the rows out
+                extra_roof = {"kv_store": (L * n_prompts * prompt_len * nkv * D * 4, L * n_prompts * prompt_len * 4 * nkv * D * 2,
+                                           L * dec_batch * nkv * D * 4, L * dec_batch * 4 * nkv * D * 2)}
             elif name == "buzarax":
                 # attention layers: every other one; full causal, q + out + the K / V rows once (prefill), the cache rows (decode)
                 La, Lr, D, nkv, Wd = (L + 1) // 2, L // 2, 128, max(1, H // 4), sz["width"]

@@ -21,7 +21,7 @@
 // token-by-token rule by rounding only.  The columns of a head's state never mix: a CTA owns 32 CPT columns of one (segment, head), a
 // warp 4 CPT of them with all their rows: lane (rg, cg) = (lane >> 2, lane & 3) holds rows 32 i + 4 rg + e (R of them) of CPT columns in
 // registers for the whole segment (neighbouring lanes read the same shared-memory words: half the cost of the other order).  Eight warps
-// own the columns, eight more HELPERS stage the next batch, make its small matrices and finish (norm, gate, store) the last one.
+// own the columns, eight (CPT = 4: four) more HELPERS stage the next batch, make its small matrices and finish (norm, gate, store) the last one.
 //
 // Single decoded tokens (hd_decode_kernel): the state is read once into registers, both products with it are summed over the CTA, the
 // update is applied and written back.
@@ -33,8 +33,8 @@
 
 namespace sllm {
 
-constexpr int HD_TOKENS = 8;               // tokens per batch, one staged by each helper warp
-constexpr int HD_WARPS = 8;                // warps of the decode kernel; warps of the prompt kernel that own columns, and its helpers
+constexpr int HD_TOKENS = 8;               // tokens per batch, shared out among the helper warps
+constexpr int HD_WARPS = 8;                // warps of the decode kernel; warps of the prompt kernel that own columns
 constexpr float HD_UNIT_EPS = 1e-6f;       // unit queries and keys (DELTA)
 constexpr float HD_DEN_EPS = 1e-6f;        // denominator (memory)
 
@@ -178,8 +178,8 @@ template <bool DELTA, int R, int CPT> constexpr int hd_prompt_smem_floats() {
            + (DELTA ? HD_TOKENS * COLS : 8 * R);                         // scaled u | n
 }
 
-__device__ __forceinline__ void hd_cta_barrier() { asm volatile("bar.sync 0, 512;" ::: "memory"); }
-__device__ __forceinline__ void hd_helper_barrier() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
+constexpr int hd_helpers(int cpt) { return cpt == 4 ? 4 : 8; }            // helper warps: few where the owners need the registers
+template <int THREADS> __device__ __forceinline__ void hd_barrier(int id) { asm volatile("bar.sync %0, %1;" ::"r"(id), "n"(THREADS) : "memory"); }
 
 // eight neighbouring floats of shared memory (16-byte aligned)
 __device__ __forceinline__ void hd_row(const float* p, float (&v)[HD_TOKENS]) {
@@ -187,10 +187,12 @@ __device__ __forceinline__ void hd_row(const float* p, float (&v)[HD_TOKENS]) {
     v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
 }
 
-// grid (segments, heads, ceil(dv / (32 CPT))), 512 threads
+// grid (segments, heads, ceil(dv / (32 CPT))), HD_WARPS + hd_helpers(CPT) warps
 template <typename T, bool DELTA, int R, int CPT>
-__global__ void __launch_bounds__(2 * HD_WARPS * 32) hd_prompt_kernel(const HeadDecayArgs p) {
+__global__ void __launch_bounds__((HD_WARPS + hd_helpers(CPT)) * 32) hd_prompt_kernel(const HeadDecayArgs p) {
     constexpr int DKP = 8 * R, P = DKP + 4, COLS = 32 * CPT, NQ = (DKP + 127) / 128;
+    constexpr int HW = hd_helpers(CPT), TPW = HD_TOKENS / HW;             // helper warps; tokens each of them takes care of: warp + HW s
+    constexpr int ALL = (HD_WARPS + HW) * 32, HELPERS = HW * 32;
     extern __shared__ __align__(16) float hd_smem[];
     float* qs = hd_smem;                                                 // [2][HD_TOKENS][P]
     float* ks = qs + 2 * HD_TOKENS * P;                                  // [2][HD_TOKENS][P]
@@ -210,156 +212,185 @@ __global__ void __launch_bounds__(2 * HD_WARPS * 32) hd_prompt_kernel(const Head
     if (n <= 0) return;
     const int seq = p.seq_ids[b], dk = p.dk, dv = p.dv, g = h / (p.H / p.G);
     const bool fresh = p.tok_pos[t0] == 0, vec = p.vec;
-    const int tid = threadIdx.x & (HD_WARPS * 32 - 1), warp = tid >> 5, lane = tid & 31;       // within the eight warps of a kind
+    const bool helper = threadIdx.x >= HD_WARPS * 32;
+    const int tid = threadIdx.x - (helper ? HD_WARPS * 32 : 0), warp = tid >> 5, lane = tid & 31;      // among the warps of its kind
     const int cta_col = blockIdx.z * COLS;
-    if (threadIdx.x >= HD_WARPS * 32) {
+    if (helper) {
         // ================ helpers
         const bool sliced = gridDim.z > 1;
         float m_run = 0.f;
         if constexpr (!DELTA) {
             const float* ns = p.nstate + ((int64_t)seq * p.H + h) * dk;
-            for (int d = tid; d < DKP; d += HD_WARPS * 32) us[d] = (!fresh && d < dk) ? ns[d] : 0.f;
+            for (int d = tid; d < DKP; d += HELPERS) us[d] = (!fresh && d < dk) ? ns[d] : 0.f;
             if (!fresh) m_run = p.mstate[(int64_t)seq * p.H + h];
         }
-        // warp w stages token w of a batch: four neighbouring entries of q and k per lane and 128, CPT neighbouring columns of v and the gate
+        // a token is staged by one warp: four neighbouring entries of q and k per lane and 128, CPT neighbouring columns of v and the gate
         const T* qp = (const T*)p.q + (int64_t)g * dk;
         const T* kp = (const T*)p.k + (int64_t)g * dk;
         const T* vp = (const T*)p.v + (int64_t)h * dv;
         const T* gp = (const T*)p.gate + (int64_t)h * dv;
         const int my_col = cta_col + lane * CPT;                             // this lane's columns while staging and finishing
-        HdRaw<T, 4> rq[NQ], rk[NQ];
-        HdRaw<T, CPT> rv, rgate;                                             // rgate: the output gate of the batch finished next
-        float fa = 0.f, fb = 0.f, nw[CPT];
+        HdRaw<T, 4> rq[TPW][NQ], rk[TPW][NQ];
+        HdRaw<T, CPT> rv[TPW], rgate[TPW];                                             // rgate: the output gate of the batch finished next
+        float fa[TPW], fb[TPW], nw[CPT];
         const float pa = p.pa[h], pb = p.pb[h];
 #pragma unroll
         for (int c = 0; c < CPT; c++) nw[c] = my_col + c < dv ? p.norm_w[h * p.norm_step + my_col + c] : 0.f;
         auto fetch = [&](int i0) {
-            const bool live = i0 + warp < n;
-            const int64_t t = t0 + (live ? i0 + warp : 0);
 #pragma unroll
-            for (int e = 0; e < NQ; e++) {
-                rq[e].load(qp + t * p.q_stride, 4 * lane + 128 * e, live ? dk : 0, vec);
-                rk[e].load(kp + t * p.k_stride, 4 * lane + 128 * e, live ? dk : 0, vec);
+            for (int s = 0; s < TPW; s++) {
+                const int tok = i0 + warp + HW * s;
+                const bool live = tok < n;
+                const int64_t t = t0 + (live ? tok : 0);
+#pragma unroll
+                for (int e = 0; e < NQ; e++) {
+                    rq[s][e].load(qp + t * p.q_stride, 4 * lane + 128 * e, live ? dk : 0, vec);
+                    rk[s][e].load(kp + t * p.k_stride, 4 * lane + 128 * e, live ? dk : 0, vec);
+                }
+                rv[s].load(vp + t * p.v_stride, my_col, live ? dv : 0, vec);
+                fa[s] = p.ga[t * p.ga_stride + h];
+                fb[s] = p.gb[t * p.gb_stride + h];
             }
-            rv.load(vp + t * p.v_stride, my_col, live ? dv : 0, vec);
-            fa = p.ga[t * p.ga_stride + h];
-            fb = p.gb[t * p.gb_stride + h];
         };
         auto fetch_gate = [&](int i0) {
-            if (!sliced && i0 >= 0 && i0 + warp < n) rgate.load(gp + (int64_t)(t0 + i0 + warp) * p.gate_stride, my_col, dv, vec);
-        };
-        // norm, gate and store of batch `i0`'s token `warp` (its read-outs are in `os`)
-        auto finish = [&](int i0) {
-            if (i0 + warp >= n) return;
-            const int64_t t = t0 + i0 + warp;
-            float o[CPT], ss = 0.f;
 #pragma unroll
-            for (int c = 0; c < CPT; c++) {
-                o[c] = os[((i0 / HD_TOKENS & 1) * HD_TOKENS + warp) * COLS + lane * CPT + c];      // columns past dv are zero
-                ss += o[c] * o[c];
+            for (int s = 0; s < TPW; s++) {
+                const int tok = i0 + warp + HW * s;
+                if (!sliced && i0 >= 0 && tok < n) rgate[s].load(gp + (int64_t)(t0 + tok) * p.gate_stride, my_col, dv, vec);
             }
-            const float f = sliced ? 1.f : rsqrtf(warp_sum(ss) / (float)dv + p.eps);
-            if (sliced) hd_put<float, CPT>(p.o_raw + (t * p.H + h) * dv, my_col, dv, vec, o);
-            else {
+        };
+        // norm, gate and store of batch `i0`'s tokens (their read-outs are in `os`)
+        auto finish = [&](int i0) {
 #pragma unroll
-                for (int c = 0; c < CPT; c++) o[c] *= f * nw[c] * hd_act<DELTA>(rgate.get(c));
+            for (int s = 0; s < TPW; s++) {
+                const int j = warp + HW * s;
+                if (i0 + j >= n) return;
+                const int64_t t = t0 + i0 + j;
+                float o[CPT], ss = 0.f;
+#pragma unroll
+                for (int c = 0; c < CPT; c++) {
+                    o[c] = os[((i0 / HD_TOKENS & 1) * HD_TOKENS + j) * COLS + lane * CPT + c];                   // columns past dv are zero
+                    ss += o[c] * o[c];
+                }
+                if (sliced) {
+                    hd_put<float, CPT>(p.o_raw + (t * p.H + h) * dv, my_col, dv, vec, o);
+                    continue;
+                }
+                const float f = rsqrtf(warp_sum(ss) / (float)dv + p.eps);
+#pragma unroll
+                for (int c = 0; c < CPT; c++) o[c] *= f * nw[c] * hd_act<DELTA>(rgate[s].get(c));
                 hd_put<T, CPT>((T*)p.out + t * p.out_stride + (int64_t)h * dv, my_col, dv, vec, o);
             }
         };
-        rgate.zero();
+#pragma unroll
+        for (int s = 0; s < TPW; s++) rgate[s].zero();
         auto prepare = [&](int i0) {                                     // stage batch i0 (fetched before), then everything but the state's part
             const int buf = (i0 / HD_TOKENS) & 1;
             float* qb = qs + buf * HD_TOKENS * P;
             float* kb = ks + buf * HD_TOKENS * P;
             float* vb = vs + buf * HD_TOKENS * COLS;
             float* sm = small + buf * HD_SMALL;
-            float fq = p.q_scale, fk = 1.f;
-            if constexpr (DELTA) {
-                float sq = 0.f, sk = 0.f;
 #pragma unroll
-                for (int e = 0; e < NQ; e++)
+            for (int s = 0; s < TPW; s++) {
+                const int tok = warp + HW * s;
+                float fq = p.q_scale, fk = 1.f;
+                if constexpr (DELTA) {
+                    float sq = 0.f, sk = 0.f;
 #pragma unroll
-                    for (int i = 0; i < 4; i++) { sq += rq[e].get(i) * rq[e].get(i); sk += rk[e].get(i) * rk[e].get(i); }
-                fq *= rsqrtf(warp_sum(sq) + HD_UNIT_EPS);
-                fk = rsqrtf(warp_sum(sk) + HD_UNIT_EPS);
+                    for (int e = 0; e < NQ; e++)
+#pragma unroll
+                        for (int i = 0; i < 4; i++) {
+                            sq += rq[s][e].get(i) * rq[s][e].get(i);
+                            sk += rk[s][e].get(i) * rk[s][e].get(i);
+                        }
+                    fq *= rsqrtf(warp_sum(sq) + HD_UNIT_EPS);
+                    fk = rsqrtf(warp_sum(sk) + HD_UNIT_EPS);
+                }
+#pragma unroll
+                for (int e = 0; e < NQ; e++) {
+                    const int d = 4 * lane + 128 * e;
+                    if (DKP % 128 != 0 && d >= DKP) break;
+                    const HdRaw<T, 4>&x = rq[s][e], &y = rk[s][e];
+                    *reinterpret_cast<float4*>(qb + tok * P + d) = make_float4(x.get(0) * fq, x.get(1) * fq, x.get(2) * fq, x.get(3) * fq);
+                    *reinterpret_cast<float4*>(kb + tok * P + d) = make_float4(y.get(0) * fk, y.get(1) * fk, y.get(2) * fk, y.get(3) * fk);
+                }
+#pragma unroll
+                for (int c = 0; c < CPT; c++) vb[tok * COLS + lane * CPT + c] = rv[s].get(c);
+                float a = 0.f, bb = DELTA ? 0.f : -INFINITY;             // past the end: no decay, nothing written
+                if (i0 + tok < n) hd_gates<DELTA>(fa[s], fb[s], pa, pb, p.cap, a, bb);
+                if (lane == 0) { gates[buf * 2 * HD_TOKENS + tok] = a; gates[(buf * 2 + 1) * HD_TOKENS + tok] = bb; }
             }
-#pragma unroll
-            for (int e = 0; e < NQ; e++) {
-                const int d = 4 * lane + 128 * e;
-                if (DKP % 128 != 0 && d >= DKP) break;
-                *reinterpret_cast<float4*>(qb + warp * P + d) = make_float4(rq[e].get(0) * fq, rq[e].get(1) * fq, rq[e].get(2) * fq, rq[e].get(3) * fq);
-                *reinterpret_cast<float4*>(kb + warp * P + d) = make_float4(rk[e].get(0) * fk, rk[e].get(1) * fk, rk[e].get(2) * fk, rk[e].get(3) * fk);
-            }
-#pragma unroll
-            for (int c = 0; c < CPT; c++) vb[warp * COLS + lane * CPT + c] = rv.get(c);
-            float a = 0.f, bb = DELTA ? 0.f : -INFINITY;                 // past the end: no decay, nothing written
-            if (i0 + warp < n) hd_gates<DELTA>(fa, fb, pa, pb, p.cap, a, bb);
-            if (lane == 0) { gates[buf * 2 * HD_TOKENS + warp] = a; gates[(buf * 2 + 1) * HD_TOKENS + warp] = bb; }
-            hd_helper_barrier();                                         // the batch is staged (memory: n is up to date)
+            hd_barrier<HELPERS>(1);                                         // the batch is staged (memory: n is up to date)
             if (i0 + HD_TOKENS < n) fetch(i0 + HD_TOKENS);               // in flight while this batch is worked on
-            // column j = `warp` of the small matrices: lane = (l, quarter of the head)
+            // the small matrices, one column j after the other: lane = (l, quarter of the head)
             const int l = lane & 7, quarter = lane >> 3;
-            float sum = 0.f, upto = 0.f, own = 0.f, floor_log = 0.f;     // own: beta of j | log input weight of l
+            float lg[HD_TOKENS], second[HD_TOKENS], own = 0.f;           // log decays; beta | running maximum; memory: log input weight of l
+            hd_row(gates + buf * 2 * HD_TOKENS, lg);
+            hd_row(gates + (buf * 2 + 1) * HD_TOKENS, second);
+            if constexpr (!DELTA) {
 #pragma unroll
-            for (int i = 0; i < HD_TOKENS; i++) {
-                const float a = gates[buf * 2 * HD_TOKENS + i], bb = gates[(buf * 2 + 1) * HD_TOKENS + i];
-                float lg = a;
-                if constexpr (DELTA) {
-                    if (i == warp) own = bb;
-                } else {
-                    const float m_new = fmaxf(a + m_run, bb);
-                    lg = a + m_run - m_new;
-                    m_run = m_new;
-                    if (i == l) own = bb - m_new;
-                    if (i == warp) floor_log = -m_new;
+                for (int i = 0; i < HD_TOKENS; i++) {
+                    const float m_new = fmaxf(lg[i] + m_run, second[i]);
+                    lg[i] += m_run - m_new;
+                    if (i == l) own = second[i] - m_new;
+                    second[i] = m_run = m_new;
                 }
-                if (i > l && i <= warp) sum += lg;
-                if (i <= warp) upto += lg;
             }
-            float kk = 0.f, kq = 0.f;
-            const float* kl = kb + l * P + quarter * (DKP / 4);
-            const float* kj = kb + warp * P + quarter * (DKP / 4);
-            const float* qj = qb + warp * P + quarter * (DKP / 4);
+#pragma unroll
+            for (int s = 0; s < TPW; s++) {
+                const int j = warp + HW * s;
+                float sum = 0.f, upto = 0.f, at_j = 0.f;
+#pragma unroll
+                for (int i = 0; i < HD_TOKENS; i++) {
+                    if (i > l && i <= j) sum += lg[i];
+                    if (i <= j) upto += lg[i];
+                    if (i == j) at_j = second[i];
+                }
+                float kk = 0.f, kq = 0.f;
+                const float* kl = kb + l * P + quarter * (DKP / 4);
+                const float* kj = kb + j * P + quarter * (DKP / 4);
+                const float* qj = qb + j * P + quarter * (DKP / 4);
 #pragma unroll 4
-            for (int i = 0; i < DKP / 4; i += 4) {
-                const float4 a = *reinterpret_cast<const float4*>(kl + i), y = *reinterpret_cast<const float4*>(qj + i);
-                kq += a.x * y.x + a.y * y.y + a.z * y.z + a.w * y.w;
+                for (int i = 0; i < DKP / 4; i += 4) {
+                    const float4 a = *reinterpret_cast<const float4*>(kl + i), y = *reinterpret_cast<const float4*>(qj + i);
+                    kq += a.x * y.x + a.y * y.y + a.z * y.z + a.w * y.w;
+                    if constexpr (DELTA) {
+                        const float4 x = *reinterpret_cast<const float4*>(kj + i);
+                        kk += a.x * x.x + a.y * x.y + a.z * x.z + a.w * x.w;
+                    }
+                }
+                kq += __shfl_xor_sync(0xffffffffu, kq, 8);
+                kq += __shfl_xor_sync(0xffffffffu, kq, 16);
                 if constexpr (DELTA) {
-                    const float4 x = *reinterpret_cast<const float4*>(kj + i);
-                    kk += a.x * x.x + a.y * x.y + a.z * x.z + a.w * x.w;
+                    kk += __shfl_xor_sync(0xffffffffu, kk, 8);
+                    kk += __shfl_xor_sync(0xffffffffu, kk, 16);
                 }
-            }
-            kq += __shfl_xor_sync(0xffffffffu, kq, 8);
-            kq += __shfl_xor_sync(0xffffffffu, kq, 16);
-            if constexpr (DELTA) {
-                kk += __shfl_xor_sync(0xffffffffu, kk, 8);
-                kk += __shfl_xor_sync(0xffffffffu, kk, 16);
-            }
-            // memory: the input weight of l joins the decay (its log may be -inf: nothing was written)
-            const float D = expf(DELTA ? sum : sum + own), d_upto = expf(upto);
-            const float m2 = l <= warp ? D * kq : 0.f;
-            float nq = 0.f;
-            if constexpr (!DELTA) {
-                for (int d = lane; d < DKP; d += 32) nq += us[d] * qb[warp * P + d];
-                nq = warp_sum(nq) * d_upto;
-                float in = m2;                                           // every quarter holds the same eight entries
-                in += __shfl_xor_sync(0xffffffffu, in, 1);
-                in += __shfl_xor_sync(0xffffffffu, in, 2);
-                in += __shfl_xor_sync(0xffffffffu, in, 4);
-                nq += in;
-            }
-            if (quarter == 0) {
-                if constexpr (DELTA) sm[M1 + l * HD_TOKENS + warp] = l < warp ? D * kk : 0.f;
-                sm[M2 + l * HD_TOKENS + warp] = m2;
-                if (warp == HD_TOKENS - 1) sm[TAIL + l] = D;
-                if (l == 0) {
-                    sm[DJ + warp] = d_upto;
-                    sm[BJ + warp] = DELTA ? own : 1.f / (fmaxf(fabsf(nq), expf(floor_log)) + HD_DEN_EPS);
+                // memory: the input weight of l joins the decay (its log may be -inf: nothing was written)
+                const float D = expf(DELTA ? sum : sum + own), d_upto = expf(upto);
+                const float m2 = l <= j ? D * kq : 0.f;
+                float nq = 0.f;
+                if constexpr (!DELTA) {
+                    for (int d = lane; d < DKP; d += 32) nq += us[d] * qb[j * P + d];
+                    nq = warp_sum(nq) * d_upto;
+                    float in = m2;                                       // every quarter holds the same eight entries
+                    in += __shfl_xor_sync(0xffffffffu, in, 1);
+                    in += __shfl_xor_sync(0xffffffffu, in, 2);
+                    in += __shfl_xor_sync(0xffffffffu, in, 4);
+                    nq += in;
+                }
+                if (quarter == 0) {
+                    if constexpr (DELTA) sm[M1 + l * HD_TOKENS + j] = l < j ? D * kk : 0.f;
+                    sm[M2 + l * HD_TOKENS + j] = m2;
+                    if (j == HD_TOKENS - 1) sm[TAIL + l] = D;
+                    if (l == 0) {
+                        sm[DJ + j] = d_upto;
+                        sm[BJ + j] = DELTA ? at_j : 1.f / (fmaxf(fabsf(nq), expf(-at_j)) + HD_DEN_EPS);
+                    }
                 }
             }
             if constexpr (!DELTA) {
-                hd_helper_barrier();                                     // every warp has read n, D(l, last) is written
-                for (int d = tid; d < DKP; d += HD_WARPS * 32) {
+                hd_barrier<HELPERS>(1);                                     // every warp has read n, D(l, last) is written
+                for (int d = tid; d < DKP; d += HELPERS) {
                     float x = us[d] * sm[DJ + HD_TOKENS - 1];
 #pragma unroll
                     for (int l = 0; l < HD_TOKENS; l++) x = fmaf(sm[TAIL + l], kb[l * P + d], x);
@@ -369,12 +400,12 @@ __global__ void __launch_bounds__(2 * HD_WARPS * 32) hd_prompt_kernel(const Head
         };
         fetch(0);
         prepare(0);
-        hd_cta_barrier();
+        hd_barrier<ALL>(0);
         for (int i0 = 0; i0 < n; i0 += HD_TOKENS) {                      // while the other warps work on batch i0
             fetch_gate(i0 - HD_TOKENS);
             if (i0 + HD_TOKENS < n) prepare(i0 + HD_TOKENS);
             if (i0 > 0) finish(i0 - HD_TOKENS);
-            hd_cta_barrier();
+            hd_barrier<ALL>(0);
         }
         const int last = (n - 1) / HD_TOKENS * HD_TOKENS;
         fetch_gate(last);
@@ -383,7 +414,7 @@ __global__ void __launch_bounds__(2 * HD_WARPS * 32) hd_prompt_kernel(const Head
             if (blockIdx.z != 0) return;
             // another CTA of this head may not have read the old n and m yet: they wait in `carry` for the head norm's launch
             float* ns = sliced ? p.carry + ((int64_t)b * p.H + h) * (dk + 1) : p.nstate + ((int64_t)seq * p.H + h) * dk;
-            for (int d = tid; d < dk; d += HD_WARPS * 32) ns[d] = us[d];
+            for (int d = tid; d < dk; d += HELPERS) ns[d] = us[d];
             if (tid == 0) *(sliced ? ns + dk : p.mstate + (int64_t)seq * p.H + h) = m_run;
         }
         return;
@@ -403,7 +434,7 @@ __global__ void __launch_bounds__(2 * HD_WARPS * 32) hd_prompt_kernel(const Head
             S[r][c].y = (!fresh && d + 1 < dk && col < dv) ? st[(int64_t)(d + 1) * dv + col] : 0.f;
         }
     }
-    hd_cta_barrier();
+    hd_barrier<ALL>(0);
     for (int i0 = 0; i0 < n; i0 += HD_TOKENS) {
         const int buf = (i0 / HD_TOKENS) & 1;
         const float* qb = qs + buf * HD_TOKENS * P;
@@ -415,45 +446,53 @@ __global__ void __launch_bounds__(2 * HD_WARPS * 32) hd_prompt_kernel(const Head
         float r[HD_TOKENS];
         int mine = 0;                                                    // which of the lane's columns r belongs to
         {
-            auto against = [&](const float* x, float (&sum)[HD_TOKENS][CPT]) {
-                float2 acc[HD_TOKENS][CPT];
+            constexpr int JH = CPT == 4 ? HD_TOKENS / 2 : HD_TOKENS;     // tokens at a time (registers)
+            float z[HD_TOKENS][CPT];
 #pragma unroll
-                for (int j = 0; j < HD_TOKENS; j++)
+            for (int j0 = 0; j0 < HD_TOKENS; j0 += JH) {
+                auto against = [&](const float* x, float (&sum)[JH][CPT]) {
+                    float2 acc[JH][CPT];
 #pragma unroll
-                    for (int c = 0; c < CPT; c++) acc[j][c] = make_float2(0.f, 0.f);
+                    for (int j = 0; j < JH; j++)
 #pragma unroll
-                for (int i = 0; i < R / 4; i++)
+                        for (int c = 0; c < CPT; c++) acc[j][c] = make_float2(0.f, 0.f);
 #pragma unroll
-                    for (int j = 0; j < HD_TOKENS; j++) {
-                        const float4 x4 = *reinterpret_cast<const float4*>(x + j * P + 32 * i + 4 * rg);
+                    for (int i = 0; i < R / 4; i++)
+#pragma unroll
+                        for (int j = 0; j < JH; j++) {
+                            const float4 x4 = *reinterpret_cast<const float4*>(x + (j0 + j) * P + 32 * i + 4 * rg);
+#pragma unroll
+                            for (int c = 0; c < CPT; c++) {
+                                acc[j][c] = fma2(S[2 * i][c], make_float2(x4.x, x4.y), acc[j][c]);
+                                acc[j][c] = fma2(S[2 * i + 1][c], make_float2(x4.z, x4.w), acc[j][c]);
+                            }
+                        }
+#pragma unroll
+                    for (int j = 0; j < JH; j++)
+#pragma unroll
+                        for (int c = 0; c < CPT; c++) sum[j][c] = acc[j][c].x + acc[j][c].y;
+                };
+                float B[JH][CPT];
+                against(qb, B);
+                if constexpr (DELTA) {                                   // even row groups take S^T k, odd ones S^T q
+                    float A[JH][CPT];
+                    against(kb, A);
+                    const bool odd = rg & 1;
+#pragma unroll
+                    for (int j = 0; j < JH; j++)
 #pragma unroll
                         for (int c = 0; c < CPT; c++) {
-                            acc[j][c] = fma2(S[2 * i][c], make_float2(x4.x, x4.y), acc[j][c]);
-                            acc[j][c] = fma2(S[2 * i + 1][c], make_float2(x4.z, x4.w), acc[j][c]);
+                            const float give = odd ? A[j][c] : B[j][c], keep = odd ? B[j][c] : A[j][c];
+                            z[j0 + j][c] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
                         }
-                    }
+                } else {
 #pragma unroll
-                for (int j = 0; j < HD_TOKENS; j++)
+                    for (int j = 0; j < JH; j++)
 #pragma unroll
-                    for (int c = 0; c < CPT; c++) sum[j][c] = acc[j][c].x + acc[j][c].y;
-            };
-            float B[HD_TOKENS][CPT];
-            against(qb, B);
-            if constexpr (DELTA) {                                       // even row groups take S^T k, odd ones S^T q
-                float A[HD_TOKENS][CPT];
-                against(kb, A);
-                const bool odd = rg & 1;
-#pragma unroll
-                for (int j = 0; j < HD_TOKENS; j++)
-#pragma unroll
-                    for (int c = 0; c < CPT; c++) {
-                        const float give = odd ? A[j][c] : B[j][c], keep = odd ? B[j][c] : A[j][c];
-                        A[j][c] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
-                    }
-                hd_reduce<1, CPT>(A, lane, mine, r);
-            } else {
-                hd_reduce<0, CPT>(B, lane, mine, r);
+                        for (int c = 0; c < CPT; c++) z[j0 + j][c] = B[j][c];
+                }
             }
+            hd_reduce<DELTA ? 1 : 0, CPT>(z, lane, mine, r);
         }
         // ---- one column per lane (several lanes hold the same one): the triangular system and the read-outs
         const int col = col_l + mine;
@@ -521,7 +560,7 @@ __global__ void __launch_bounds__(2 * HD_WARPS * 32) hd_prompt_kernel(const Head
                 }
             }
         }
-        hd_cta_barrier();                                                // the next batch is prepared, `ob` is written
+        hd_barrier<ALL>(0);                                                // the next batch is prepared, `ob` is written
     }
 #pragma unroll
     for (int r = 0; r < R / 2; r++) {
@@ -737,7 +776,7 @@ template <typename T, bool DELTA, int R, int CPT> static int hd_launch_prompt(co
     auto kern = hd_prompt_kernel<T, DELTA, R, CPT>;
     const size_t smem = sizeof(float) * hd_prompt_smem_floats<DELTA, R, CPT>();
     if (first_use_on_this_device(attr_mask)) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    kern<<<dim3((unsigned)a.num_segs, (unsigned)a.H, (unsigned)cdiv(a.dv, 32 * CPT)), 2 * HD_WARPS * 32, smem, stream>>>(a);
+    kern<<<dim3((unsigned)a.num_segs, (unsigned)a.H, (unsigned)cdiv(a.dv, 32 * CPT)), (HD_WARPS + hd_helpers(CPT)) * 32, smem, stream>>>(a);
     return cdiv(a.dv, 32 * CPT);
 }
 
@@ -746,7 +785,8 @@ template <typename T, bool DELTA> static int hd_prompt(const HeadDecayArgs& a, i
     const int rows = cdiv(a.dk, 8);
     if (rows <= 8)
         return want >= 4 ? hd_launch_prompt<T, DELTA, 8, 4>(a, s) : want >= 2 ? hd_launch_prompt<T, DELTA, 8, 2>(a, s) : hd_launch_prompt<T, DELTA, 8, 1>(a, s);
-    if (rows <= 16) return want >= 2 ? hd_launch_prompt<T, DELTA, 16, 2>(a, s) : hd_launch_prompt<T, DELTA, 16, 1>(a, s);
+    if (rows <= 16)
+        return want >= 4 ? hd_launch_prompt<T, DELTA, 16, 4>(a, s) : want >= 2 ? hd_launch_prompt<T, DELTA, 16, 2>(a, s) : hd_launch_prompt<T, DELTA, 16, 1>(a, s);
     if (rows <= 32) return hd_launch_prompt<T, DELTA, 32, 1>(a, s);
     return hd_launch_prompt<T, DELTA, 64, 1>(a, s);
 }

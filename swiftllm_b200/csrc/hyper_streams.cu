@@ -42,7 +42,7 @@ template <typename T> struct HsVec<T, 4> {
 // (one_stream).  y null: the streams stay as they are.  x_out (may be x_in, unless one_stream) null: not written.  h null: no read.
 // SMAX: streams held in registers (S <= SMAX); V entries a thread and turn.  Dynamic shared memory: width floats.
 template <typename T, int SMAX, int V>
-__global__ void __launch_bounds__(256) stream_mix_norm_kernel(const float* x_in, int one_stream, int S, const T* __restrict__ y,
+__global__ void __launch_bounds__(256, SMAX <= 4 ? 4 : 1) stream_mix_norm_kernel(const float* x_in, int one_stream, int S, const T* __restrict__ y,
                                                               const float* __restrict__ mix, const float* __restrict__ share,
                                                               const float* __restrict__ in, const float* __restrict__ norm_w,
                                                               float eps, float* x_out, T* __restrict__ h,

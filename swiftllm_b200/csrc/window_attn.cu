@@ -148,8 +148,8 @@ __global__ void __launch_bounds__(128) shared_kv_store_kernel(
 // Queries and keys that are RMS-normed over their WHOLE projection (all heads together, weights qw [H * dk], kw [G * dk]) and then turned
 // on their first rot entries, with the un-normed keys as values: one CTA per token writes the cache row (shared_kv with krot = rot, see
 // the top of the file) and the queries in the order the attention kernels read them.  Both rows wait in shared memory as fp32
-// ((H + G) dk floats) between the sums and the writes; then a warp takes a head at a time.  VEC: eight entries a load (rows aligned,
-// H dk and G dk multiples of 8) and two a store (dk even).
+// ((H + G) dk floats, with the token's angles behind them) between the sums and the writes; then a warp takes a head at a time.  VEC: 16 bytes a load (rows aligned)
+// and four entries a store (dk and rot multiples of 4).
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) whole_norm_rope_store_kernel(
     const T* __restrict__ q, int64_t q_stride, const T* __restrict__ k, int64_t k_stride, const float* __restrict__ qw,
@@ -158,7 +158,7 @@ __global__ void __launch_bounds__(256) whole_norm_rope_store_kernel(
     T* __restrict__ cache, int n_slots, int slot, int block_size, T* __restrict__ q_out, int H, int G, int dk, int rot, int halves) {
     extern __shared__ __align__(16) float smem[];
     __shared__ float red[32];
-    constexpr int N = VEC ? 2 : 1;
+    constexpr int N = VEC ? 4 : 1;
     const int64_t t = blockIdx.x;
     float* qs = smem;                          // [H * dk]
     float* ks = qs + H * dk;                   // [G * dk]
@@ -166,8 +166,10 @@ __global__ void __launch_bounds__(256) whole_norm_rope_store_kernel(
     const int blk = block_table[(int64_t)tok_seq[t] * max_blocks_per_seq + pos / block_size];
     const int koff = shared_kv_key_offset(G), kw_cols = dk + rot, hq = H / G, pass = dk - rot;
     T* dst = cache + (((int64_t)blk * n_slots + slot) * block_size + pos % block_size) * shared_kv_row(G, kw_cols);
-    const float* cs = cosb != nullptr ? cosb + t * (rot >> 1) : nullptr;
-    const float* sn = sinb != nullptr ? sinb + t * (rot >> 1) : nullptr;
+    const int half = rot >> 1;
+    float* cs = ks + G * dk;                   // [half] each
+    float* sn = cs + half;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) { cs[i] = cosb[t * half + i]; sn[i] = sinb[t * half + i]; }
     auto stage = [&](const T* src, float* to, int n) {
         float ss = 0.f;
         if constexpr (VEC) {
@@ -188,15 +190,20 @@ __global__ void __launch_bounds__(256) whole_norm_rope_store_kernel(
         return ss;
     };
     const float sq = stage(q + t * q_stride, qs, H * dk), sk = stage(k + t * k_stride, ks, G * dk);
-    const float qinv = 1.f / sqrtf(block_sum(sq, red) / (float)(H * dk) + eps);
-    const float kinv = 1.f / sqrtf(block_sum(sk, red) / (float)(G * dk) + eps);          // (both rows are staged)
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5, half = rot >> 1;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
+    const float wq = warp_sum(sq), wk_ = warp_sum(sk);
+    if (lane == 0) { red[warp] = wq; red[16 + warp] = wk_; }
+    __syncthreads();                                                     // both rows, the angles and the warps' sums are staged
+    float q2 = 0.f, k2 = 0.f;
+    for (int w = 0; w < nwarps; w++) { q2 += red[w]; k2 += red[16 + w]; }
+    const float qinv = 1.f / sqrtf(q2 / (float)(H * dk) + eps), kinv = 1.f / sqrtf(k2 / (float)(G * dk) + eps);
     for (int g = threadIdx.x; g < G; g += blockDim.x) reinterpret_cast<float*>(dst)[g] = kinv;
     auto put = [&](T* to, const float* v) {                              // N neighbouring entries
         if constexpr (VEC) {
-            struct alignas(2 * sizeof(T)) Pair { T e[2]; } x;
-            stf(x.e, v[0]); stf(x.e + 1, v[1]);
-            *reinterpret_cast<Pair*>(to) = x;
+            struct alignas(4 * sizeof(T)) Pack { T e[4]; } x;
+#pragma unroll
+            for (int e = 0; e < 4; e++) stf(x.e + e, v[e]);
+            *reinterpret_cast<Pack*>(to) = x;
         } else {
             stf(to, v[0]);
         }
@@ -1214,11 +1221,11 @@ int sllm_whole_norm_rope_store(const void* q, int64_t q_row_stride, const void* 
     if (num_tokens == 0) return 0;
     SLLM_REQUIRE(q && k && q_norm_w && k_norm_w && tok_seq && tok_pos && block_table && cache && q_out && (rot_dims == 0 || (cosb && sinb)),
                  "whole_norm_rope_store: null pointer");
-    const size_t smem = (size_t)(num_heads + num_kv_heads) * dk * sizeof(float);
+    const size_t smem = ((size_t)(num_heads + num_kv_heads) * dk + rot_dims) * sizeof(float);
     SLLM_REQUIRE(smem <= 200 * 1024, "whole_norm_rope_store: %d + %d heads of %d entries do not fit in shared memory", num_heads,
                  num_kv_heads, dk);
     const int per = dtype == SLLM_F32 ? 4 : 8;
-    const bool vec = dk % 2 == 0 && (num_heads * dk) % per == 0 && (num_kv_heads * dk) % per == 0 && q_row_stride % per == 0 &&
+    const bool vec = dk % 4 == 0 && rot_dims % 4 == 0 && (num_heads * dk) % per == 0 && (num_kv_heads * dk) % per == 0 && q_row_stride % per == 0 &&
                      k_row_stride % per == 0 && (((uintptr_t)q | (uintptr_t)k | (uintptr_t)q_out | (uintptr_t)cache) & 15) == 0;
     SLLM_DISPATCH_DTYPE_F32(dtype, {
         static unsigned long long attr_mask = 0;
